@@ -270,13 +270,13 @@ __device__ __forceinline__ float rotated(const float* x, int d, int rd, int neig
 // null), rotation of their first rd dimensions (inv_freq or null), q -> q_out [T, Hq, hd]; k, v -> pages
 // [Hkv, num_pages, page_size, hd] and [Hv, .., vd].  Grid (T, Hq + Hkv + Hv) (or (T, Hq) when nothing is written).
 // bias: one entry per column of a row, added to the summed slices, or null.  v_is_k: the rows hold no v heads; a value is its
-// key as projected (bias included, before norm and rotation).
+// key as projected (bias included, before norm and rotation).  v_norm: a value is divided by its root mean square (no weight).
 template <typename T>
 __global__ void __launch_bounds__(128) qkv_pages_kernel(const float* qkv, int ld, int splits, size_t split_stride, int Hq, int Hkv, int hd, int vd,
                                                         const float* q_norm, const float* k_norm, float eps, const float* inv_freq, int rd,
                                                         int neighbours, const int* positions, const int* req_of_token,
                                                         const int* block_table, int max_blocks, int page_size, int num_pages, T* q_out,
-                                                        T* k_pages, T* v_pages, int Hv, const float* bias, int v_is_k) {
+                                                        T* k_pages, T* v_pages, int Hv, const float* bias, int v_is_k, int v_norm) {
     pdl_enter();
     extern __shared__ float xs[];            // max(hd, vd) floats
     __shared__ float red[32];
@@ -298,9 +298,9 @@ __global__ void __launch_bounds__(128) qkv_pages_kernel(const float* qkv, int ld
         ss = fmaf(v, v, ss);
     }
     const float* nw = kind == 0 ? q_norm : kind == 1 ? k_norm : nullptr;
-    if (nw) {
+    if (nw || (kind == 2 && v_norm)) {
         const float inv = rsqrtf(block_sum(ss, red) / (float)n + eps);
-        for (int d = threadIdx.x; d < n; d += blockDim.x) xs[d] = xs[d] * inv * nw[d];
+        for (int d = threadIdx.x; d < n; d += blockDim.x) xs[d] = xs[d] * inv * (nw ? nw[d] : 1.0f);
     }
     __syncthreads();
     T* dst;
@@ -325,7 +325,7 @@ __global__ void __launch_bounds__(256) qkv_pages_warp_kernel(const float* qkv, i
                                                              const float* q_norm, const float* k_norm, float eps, const float* inv_freq, int rd,
                                                              int neighbours, const int* positions, const int* req_of_token,
                                                              const int* block_table, int max_blocks, int page_size, int num_pages, T* q_out,
-                                                             T* k_pages, T* v_pages, int heads, const float* bias, int v_is_k) {
+                                                             T* k_pages, T* v_pages, int heads, const float* bias, int v_is_k, int v_norm) {
     pdl_enter();
     __shared__ float stage[8][256];
     const int t = blockIdx.x, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
@@ -354,12 +354,12 @@ __global__ void __launch_bounds__(256) qkv_pages_warp_kernel(const float* qkv, i
         ss = fmaf(v, v, ss);
     }
     const float* nw = kind == 0 ? q_norm : kind == 1 ? k_norm : nullptr;
-    if (nw) {
+    if (nw || (kind == 2 && v_norm)) {
         const float inv = rsqrtf(warp_sum(ss) / (float)n + eps);
 #pragma unroll
         for (int j = 0; j < 8; ++j) {
             const int d = lane + 32 * j;
-            if (d < n) x[j] = x[j] * inv * nw[d];
+            if (d < n) x[j] = x[j] * inv * (nw ? nw[d] : 1.0f);
         }
     }
     T* dst;
@@ -399,9 +399,9 @@ __global__ void __launch_bounds__(256) qkv_pages_warp_kernel(const float* qkv, i
 // last rd values, the first `turn` of them rotated -> qr[(h T + t) rd].  Block (t, H): the latent, RMS-normed with weight
 // cw -> the page row's first `rank` values; the shared rotated key part -> the row's last rd.  neighbours: the rotation
 // pairs 2i with 2i+1 instead of i with i + turn/2.  A layer that reads another layer's pages has no block (t, H) (and x no
-// latent columns).
+// latent columns).  The latent (and the shared key part after it) is read from rows of its own: xc + t ldc.
 template <typename T>
-__global__ void __launch_bounds__(128) latent_prep_kernel(const float* x, int ld, int H, int dim, int rd, int rank, const float* cw, float eps,
+__global__ void __launch_bounds__(128) latent_prep_kernel(const float* x, int ld, const float* xc, int ldc, int H, int dim, int rd, int rank, const float* cw, float eps,
                                                           const float* inv_freq, int turn, int neighbours, const int* positions,
                                                           const int* req_of_token, const int* block_table, int max_blocks, int page_size,
                                                           T* qn, T* qr, T* pages, int T_) {
@@ -418,7 +418,7 @@ __global__ void __launch_bounds__(128) latent_prep_kernel(const float* x, int ld
         for (int d = threadIdx.x; d < rd; d += blockDim.x) qr[row * rd + d] = from_f32<T>(rotated(xs, d, turn, neighbours, pos, inv_freq));
         return;
     }
-    const float* src = x + (size_t)t * ld + (size_t)H * (dim + rd);
+    const float* src = xc + (size_t)t * ldc;
     float ss = 0.0f;
     for (int d = threadIdx.x; d < rank; d += blockDim.x) ss = fmaf(src[d], src[d], ss);
     const float inv = rsqrtf(block_sum(ss, red) / (float)rank + eps);
@@ -462,7 +462,62 @@ __global__ void __launch_bounds__(128) map_difference_kernel(const float* a, T* 
     for (int d = lane; d < dv; d += 32) out[(size_t)row * dv + d] = from_f32<T>((a1[d] - lambda * a2[d]) * inv);
 }
 
+// Every head's result times the sigmoid of its number: a [T, H, n] in the storage type, in place; the numbers are columns
+// col .. col + H of p, FP32 [slices, T, ld], the slices added in order.  A warp per (token, head).
+template <typename T>
+__global__ void __launch_bounds__(128) gate_heads_kernel(T* a, const float* p, int slices, size_t slice_stride, int ld, int col, int rows, int H, int n) {
+    pdl_enter();
+    const int row = blockIdx.x * 4 + (threadIdx.x >> 5), lane = threadIdx.x & 31;
+    if (row >= rows) return;
+    const float* src = p + (size_t)(row / H) * ld + col + row % H;
+    float z = src[0];
+    for (int s = 1; s < slices; ++s) z += src[s * slice_stride];
+    const float g = 1.0f / (1.0f + expf(-z));
+    T* mine = a + (size_t)row * n;
+    for (int d = lane; d < n; d += 32) mine[d] = from_f32<T>(to_f32(mine[d]) * g);
+}
+
+// out[t] = T(x[t, col : col + n] over its root mean square times w): n columns of FP32 rows, normed on their own.  A block per row.
+template <typename T>
+__global__ void __launch_bounds__(128) norm_columns_kernel(const float* x, int ld, int col, int n, const float* w, float eps, T* out) {
+    pdl_enter();
+    __shared__ float red[32];
+    const float* src = x + (size_t)blockIdx.x * ld + col;
+    constexpr int KEEP = 8;                    // entries a thread keeps between the two passes; wider rows are read again
+    float v[KEEP], ss = 0.0f;
+#pragma unroll
+    for (int j = 0; j < KEEP; ++j) {
+        const int d = threadIdx.x + 128 * j;
+        v[j] = d < n ? src[d] : 0.0f;
+        ss = fmaf(v[j], v[j], ss);
+    }
+    for (int d = threadIdx.x + 128 * KEEP; d < n; d += 128) ss = fmaf(src[d], src[d], ss);
+    const float inv = rsqrtf(block_sum(ss, red) / (float)n + eps);
+    T* dst = out + (size_t)blockIdx.x * n;
+#pragma unroll
+    for (int j = 0; j < KEEP; ++j) {
+        const int d = threadIdx.x + 128 * j;
+        if (d < n) dst[d] = from_f32<T>(v[j] * inv * w[d]);
+    }
+    for (int d = threadIdx.x + 128 * KEEP; d < n; d += 128) dst[d] = from_f32<T>(src[d] * inv * w[d]);
+}
+
 }  // namespace
+
+Q6K_API int q6k_gate_heads(void* a, const float* p, int slices, long long slice_stride, int ld, int col, int T_, int H, int n, int dtype, cudaStream_t st) {
+    if (T_ == 0) return 0;
+    Q6K_REQUIRE(T_ > 0 && H > 0 && n > 0 && slices >= 1 && col >= 0 && col + H <= ld && (long long)T_ * H <= 0x7fffffffLL, "gate_heads: bad sizes T=%d H=%d n=%d", T_, H, n);
+    Q6K_DISPATCH(dtype, q6k_launch(gate_heads_kernel<T>, dim3((unsigned)(((long long)T_ * H + 3) / 4)), 128, 0, st, (T*)a, p, slices, (size_t)slice_stride, ld, col,
+                                   T_ * H, H, n););
+    return q6k_check_launch("gate_heads");
+}
+
+Q6K_API int q6k_norm_columns(const float* x, int ld, int col, int n, const float* w, float eps, void* out, int T_, int dtype, cudaStream_t st) {
+    if (T_ == 0) return 0;
+    Q6K_REQUIRE(T_ > 0 && n > 0 && col >= 0 && col + n <= ld && w, "norm_columns: bad sizes T=%d n=%d", T_, n);
+    Q6K_DISPATCH(dtype, q6k_launch(norm_columns_kernel<T>, dim3(T_), 128, 0, st, x, ld, col, n, w, eps, (T*)out););
+    return q6k_check_launch("norm_columns");
+}
 
 Q6K_API int q6k_map_difference(const float* a, void* out, int T_, int H, int dv, float lambda, float eps, float mult, int dtype, cudaStream_t st) {
     if (T_ == 0) return 0;
@@ -514,7 +569,7 @@ Q6K_API int q6k_qkv_pages(const float* qkv, int ld, int splits, long long split_
                           const float* q_norm, const float* k_norm, float eps, const float* inv_freq, int rotary_dim, int neighbours,
                           const int* positions, const int* req_of_token, const int* block_table, int max_blocks, int page_size,
                           int num_pages, void* q_out, void* k_pages, void* v_pages, int write_kv, int dtype, int Hv, const float* bias, int v_is_k,
-                          cudaStream_t st) {
+                          int v_norm, cudaStream_t st) {
     if (T_ == 0) return 0;
     if (Hv <= 0) Hv = Hkv;
     Q6K_REQUIRE(!v_is_k || (Hv == Hkv && vd == hd), "qkv_pages: values that are the keys have the keys' heads and width");
@@ -528,24 +583,24 @@ Q6K_API int q6k_qkv_pages(const float* qkv, int ld, int splits, long long split_
     if (hd <= 256 && vd <= 256 && (heads + 7) / 8 <= 65535) {                 // narrow heads: a warp per head
         Q6K_DISPATCH(dtype, q6k_launch(qkv_pages_warp_kernel<T>, dim3(T_, (heads + 7) / 8), 256, 0, st, qkv, ld, splits, (size_t)split_stride, Hq, Hkv,
                                        hd, vd, q_norm, k_norm, eps, inv_freq, inv_freq ? rotary_dim : 0, neighbours, positions, req_of_token,
-                                       block_table, max_blocks, page_size, num_pages, (T*)q_out, (T*)k_pages, (T*)v_pages, heads, bias, v_is_k););
+                                       block_table, max_blocks, page_size, num_pages, (T*)q_out, (T*)k_pages, (T*)v_pages, heads, bias, v_is_k, v_norm););
         return q6k_check_launch("qkv_pages");
     }
     Q6K_DISPATCH(dtype, q6k_launch(qkv_pages_kernel<T>, dim3(T_, heads), 128, smem, st, qkv, ld, splits, (size_t)split_stride, Hq, Hkv, hd, vd,
                                    q_norm, k_norm, eps, inv_freq, inv_freq ? rotary_dim : 0, neighbours, positions, req_of_token, block_table,
-                                   max_blocks, page_size, num_pages, (T*)q_out, (T*)k_pages, (T*)v_pages, Hv, bias, v_is_k););
+                                   max_blocks, page_size, num_pages, (T*)q_out, (T*)k_pages, (T*)v_pages, Hv, bias, v_is_k, v_norm););
     return q6k_check_launch("qkv_pages");
 }
 
-Q6K_API int q6k_latent_prep(const float* x, int ld, int T_, int H, int dim, int rd, int rank, const float* cw, float eps,
+Q6K_API int q6k_latent_prep(const float* x, int ld, const float* xc, int ldc, int T_, int H, int dim, int rd, int rank, const float* cw, float eps,
                             const float* inv_freq, int turn, int neighbours, const int* positions, const int* req_of_token,
                             const int* block_table, int max_blocks, int page_size, void* qn, void* qr, void* pages, int dtype, cudaStream_t st) {
     if (T_ == 0) return 0;
-    Q6K_REQUIRE(T_ > 0 && H > 0 && dim > 0 && rd >= 0 && (rank > 0 || !pages), "latent_prep: bad sizes T=%d H=%d dim=%d rd=%d rank=%d", T_, H, dim, rd, rank);
+    Q6K_REQUIRE(T_ > 0 && H > 0 && dim > 0 && rd >= 0 && ((rank > 0 && xc) || !pages), "latent_prep: bad sizes T=%d H=%d dim=%d rd=%d rank=%d", T_, H, dim, rd, rank);
     Q6K_REQUIRE(turn >= 0 && turn % 2 == 0 && turn <= rd && (turn == 0 || inv_freq), "latent_prep: %d turning dimensions of %d", turn, rd);
     Q6K_REQUIRE(H + 1 <= 65535 && (!pages || (page_size > 0 && max_blocks > 0 && cw)), "latent_prep: bad grid or pages");
     const size_t smem = (size_t)(rd > 0 ? rd : 1) * sizeof(float);
-    Q6K_DISPATCH(dtype, q6k_launch(latent_prep_kernel<T>, dim3(T_, pages ? H + 1 : H), 128, smem, st, x, ld, H, dim, rd, rank, cw, eps, inv_freq, turn,
+    Q6K_DISPATCH(dtype, q6k_launch(latent_prep_kernel<T>, dim3(T_, pages ? H + 1 : H), 128, smem, st, x, ld, xc, ldc, H, dim, rd, rank, cw, eps, inv_freq, turn,
                                    neighbours, positions, req_of_token, block_table, max_blocks, page_size, (T*)qn, (T*)qr, (T*)pages, T_););
     return q6k_check_launch("latent_prep");
 }

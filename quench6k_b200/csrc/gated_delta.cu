@@ -364,15 +364,17 @@ __global__ void __launch_bounds__(DELTA_THREADS) gated_delta_kernel(const float*
 }
 
 // grid (T, ceil(H / 4)), a warp per (token, head): out = T(o / rms(o) * w * silu(gate)).  Heads up to 256 wide keep their
-// values and gates in registers, all loads asked for before the sum; wider ones read the row twice.
+// values and gates in registers, all loads asked for before the sum; wider ones read the row twice.  w_stride: floats from a
+// head's weights to the next head's (0: shared by the heads).
 template <typename T>
-__global__ void __launch_bounds__(128) delta_out_kernel(const float* o, const float* p, int ldp, int g_col, const float* w, float eps, T* out,
+__global__ void __launch_bounds__(128) delta_out_kernel(const float* o, const float* p, int ldp, int g_col, const float* w, int w_stride, float eps, T* out,
                                                         int H, int dv, int gate) {
     pdl_enter();
     const int t = blockIdx.x, head = blockIdx.y * 4 + (threadIdx.x >> 5), lane = threadIdx.x & 31;
     if (head >= H) return;
     const float* orow = o + ((size_t)t * H + head) * dv;
     const float* grow = p + (size_t)t * ldp + g_col + head * dv;
+    w += (size_t)head * w_stride;
     T* dst = out + ((size_t)t * H + head) * dv;
     if (dv <= 256) {
         float v[8], g[8], ww[8];
@@ -493,7 +495,7 @@ Q6K_API int q6k_gated_delta(float* u, int ldu, const float* p, int ldp, int b_co
 }
 
 Q6K_API int q6k_delta_out(const float* o, const float* p, int ldp, int g_col, const float* w, float eps, void* out, int T_, int H, int dv, int dtype,
-                          int gate, cudaStream_t st) {
+                          int gate, int w_stride, cudaStream_t st) {
     if (T_ == 0) return 0;
     Q6K_REQUIRE(T_ > 0 && H > 0 && dv > 0 && (gate == 0 || gate == 1), "delta_out: bad sizes T=%d H=%d dv=%d gate=%d", T_, H, dv, gate);
     Q6K_REQUIRE((H + 3) / 4 <= 65535, "delta_out: %d heads exceed the grid limit", H);
@@ -501,6 +503,6 @@ Q6K_API int q6k_delta_out(const float* o, const float* p, int ldp, int g_col, co
         Q6K_DISPATCH(dtype, q6k_launch(delta_out_row_kernel<T>, dim3(T_), 256, 0, st, o, p, ldp, g_col, w, eps, (T*)out, dv, gate););
         return q6k_check_launch("delta_out");
     }
-    Q6K_DISPATCH(dtype, q6k_launch(delta_out_kernel<T>, dim3(T_, (H + 3) / 4), 128, 0, st, o, p, ldp, g_col, w, eps, (T*)out, H, dv, gate););
+    Q6K_DISPATCH(dtype, q6k_launch(delta_out_kernel<T>, dim3(T_, (H + 3) / 4), 128, 0, st, o, p, ldp, g_col, w, w_stride, eps, (T*)out, H, dv, gate););
     return q6k_check_launch("delta_out");
 }

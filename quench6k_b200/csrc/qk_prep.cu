@@ -1,4 +1,4 @@
-// Per-head RMSNorm of q and k, rotary position encoding, q into the operand dtype and k, v into
+// Per-head RMSNorm of q and k (and, on request, of v without a weight), rotary position encoding, q into the operand dtype and k, v into
 // the pages of the cache.  Reference: crates/cuda/kernels/flint.cu:125-173 (there for one
 // sequence, a contiguous cache, head size 128 and theta 10000 compiled in).
 //
@@ -21,7 +21,7 @@ template <typename T>
 __global__ void qk_prep_kernel(const float* qkv, int ld, int splits, size_t split_stride, int Hq, int Hkv, int hd, const float* q_norm, const float* k_norm,
                                float eps, const float* inv_freq, int rd, int neighbours, const int* positions, const int* req_of_token,
                                const int* block_table, int max_blocks, int page_size, int num_pages, T* q_out, T* k_pages, T* v_pages,
-                               const float* bias, int v_is_k) {
+                               const float* bias, int v_is_k, int v_norm) {
     pdl_enter();
     extern __shared__ float xs[];            // hd floats
     __shared__ float red[32];
@@ -54,21 +54,25 @@ __global__ void qk_prep_kernel(const float* qkv, int ld, int splits, size_t spli
             x = first ? xs[d] * cs - xs[partner] * sn : xs[d] * cs + xs[partner] * sn;
         }
     }
+    float v = projected;
+    const int kh = h - Hq;
+    if (!is_q && !v_is_k && live) {
+        v = 0.0f;
+        for (int s = 0; s < splits; ++s) v += qkv[s * split_stride + (size_t)t * ld + (size_t)(Hq + Hkv + kh) * hd + d];
+        if (bias) v += bias[(size_t)(Hq + Hkv + kh) * hd + d];
+    }
+    if (!is_q && v_norm) {                   // a value over its root mean square
+        const float ss = block_sum(live ? v * v : 0.0f, red);
+        v *= rsqrtf(ss / (float)hd + eps);
+    }
     if (!live) return;
     if (is_q) {
         q_out[((size_t)t * Hq + h) * hd + d] = from_f32<T>(x);
     } else {
-        const int kh = h - Hq;
         const int page = block_table[(size_t)req_of_token[t] * max_blocks + pos / page_size];
         if (page < 0) return;                 // no page behind this position: nothing is written
         const size_t row = (((size_t)kh * num_pages + page) * page_size + pos % page_size) * hd + d;
         k_pages[row] = from_f32<T>(x);
-        float v = projected;
-        if (!v_is_k) {
-            v = 0.0f;
-            for (int s = 0; s < splits; ++s) v += qkv[s * split_stride + (size_t)t * ld + (size_t)(Hq + Hkv + kh) * hd + d];
-            if (bias) v += bias[(size_t)(Hq + Hkv + kh) * hd + d];
-        }
         v_pages[row] = from_f32<T>(v);
     }
 }
@@ -83,7 +87,7 @@ __global__ void __launch_bounds__(256) qk_prep_warp_kernel(const float* qkv, int
                                                            const float* k_norm, float eps, const float* inv_freq, int rd, int neighbours,
                                                            const int* positions, const int* req_of_token, const int* block_table,
                                                            int max_blocks, int page_size, int num_pages, T* q_out, T* k_pages,
-                                                           T* v_pages, int heads, const float* bias, int v_is_k) {
+                                                           T* v_pages, int heads, const float* bias, int v_is_k, int v_norm) {
     pdl_enter();
     constexpr int hd = EPL * 32, half = hd / 2;
     __shared__ float rot_cos[half], rot_sin[half];
@@ -171,6 +175,14 @@ __global__ void __launch_bounds__(256) qk_prep_warp_kernel(const float* qkv, int
 #pragma unroll
         for (int i = 0; i < EPL; ++i) dst[lane + 32 * i] = from_f32<T>(x[i]);
     } else {
+        if (v_norm) {                                                    // a value over its root mean square
+            float sv = 0.0f;
+#pragma unroll
+            for (int i = 0; i < EPL; ++i) sv = fmaf(v[i], v[i], sv);
+            const float inv = rsqrtf(warp_sum(sv) / (float)hd + eps);
+#pragma unroll
+            for (int i = 0; i < EPL; ++i) v[i] *= inv;
+        }
         if (page < 0) return;
         const size_t row = (((size_t)kh * num_pages + page) * page_size + pos % page_size) * hd;
 #pragma unroll
@@ -190,11 +202,12 @@ __global__ void __launch_bounds__(256) qk_prep_warp_kernel(const float* qkv, int
 // write_kv == 0: only q is produced (the layer reads a cache another layer wrote).
 // splits > 1: qkv is [splits, T, ld] (slices split_stride floats apart) and the slices are summed in order first.
 // bias: FP32, one entry per column of a row (q, k, v side by side), added to the summed slices, or null.  v_is_k: a key's value
-// is the key itself as projected (bias included, before norm and rotation); the rows then hold no v heads.
+// is the key itself as projected (bias included, before norm and rotation); the rows then hold no v heads.  v_norm: a value is
+// divided by its root mean square (eps as the norms'), no weight, before it is stored.
 Q6K_API int q6k_qk_prep(const float* qkv, int ld, int splits, long long split_stride, int T_, int Hq, int Hkv, int hd, const float* q_norm, const float* k_norm,
                         float eps, const float* inv_freq, int rotary_dim, int neighbours, const int* positions, const int* req_of_token,
                         const int* block_table, int max_blocks, int page_size, int num_pages, void* q_out, void* k_pages,
-                        void* v_pages, int write_kv, int dtype, const float* bias, int v_is_k, cudaStream_t st) {
+                        void* v_pages, int write_kv, int dtype, const float* bias, int v_is_k, int v_norm, cudaStream_t st) {
     if (T_ == 0) return 0;
     Q6K_REQUIRE(T_ > 0 && Hq > 0 && Hkv > 0 && hd > 0, "qk_prep: bad sizes T=%d Hq=%d Hkv=%d hd=%d", T_, Hq, Hkv, hd);
     Q6K_REQUIRE(splits >= 1, "qk_prep: bad split count %d", splits);
@@ -208,7 +221,7 @@ Q6K_API int q6k_qk_prep(const float* qkv, int ld, int splits, long long split_st
         Q6K_REQUIRE(wgrid.y <= 65535, "qk_prep: %d heads exceed the grid limit", heads);
 #define WARP_LAUNCH(EPL)                                                                                                    \
     q6k_launch(qk_prep_warp_kernel<T, EPL>, wgrid, 256, 0, st, qkv, ld, splits, (size_t)split_stride, Hq, Hkv, q_norm, k_norm, eps, inv_freq, rd, neighbours, positions, req_of_token, \
-                                                       block_table, max_blocks, page_size, num_pages, (T*)q_out, (T*)k_pages, (T*)v_pages, heads, bias, v_is_k)
+                                                       block_table, max_blocks, page_size, num_pages, (T*)q_out, (T*)k_pages, (T*)v_pages, heads, bias, v_is_k, v_norm)
         Q6K_DISPATCH(dtype, {
             if (hd == 64) WARP_LAUNCH(2);
             else if (hd == 128) WARP_LAUNCH(4);
@@ -221,6 +234,6 @@ Q6K_API int q6k_qk_prep(const float* qkv, int ld, int splits, long long split_st
     dim3 grid(T_, heads);
     Q6K_DISPATCH(dtype, q6k_launch(qk_prep_kernel<T>, grid, threads, hd * sizeof(float), st, 
                             qkv, ld, splits, (size_t)split_stride, Hq, Hkv, hd, q_norm, k_norm, eps, inv_freq, rd, neighbours, positions, req_of_token, block_table,
-                            max_blocks, page_size, num_pages, (T*)q_out, (T*)k_pages, (T*)v_pages, bias, v_is_k););
+                            max_blocks, page_size, num_pages, (T*)q_out, (T*)k_pages, (T*)v_pages, bias, v_is_k, v_norm););
     return q6k_check_launch("qk_prep");
 }

@@ -124,33 +124,39 @@ __global__ void __launch_bounds__(256) scaled_add_norm4_kernel(float* h, const f
     }
 }
 
-// act: 0 silu, 1 the tanh form of gelu, 2 the square of relu
+// act: 0 silu, 1 the tanh form of gelu, 2 the square of relu, 3 tanh
 __device__ __forceinline__ float activation(float z, int act) {
     if (act == 0) return z / (1.0f + expf(-z));
     if (act == 1) return 0.5f * z * (1.0f + tanhf(0.7978845608028654f * (z + 0.044715f * z * z * z)));
+    if (act == 3) return tanhf(z);
     const float p = fmaxf(z, 0.0f);
     return p * p;
 }
 
-// out[r, i] = T(act(x[r, i]) * x[r, I + i]) (gated: x has 2 I columns) or T(act(x[r, i])).
+// out[r, i] = T(act(x[r, i]) * x[r, I + i]) (gated: x has 2 I columns) or T(act(x[r, i])); x may be split-K slices, added in order.
 template <typename T>
-__global__ void activate_kernel(const float* x, int ldx, T* out, int I, size_t count, int gated, int act) {
+__global__ void activate_kernel(const float* x, int slices, size_t slice_stride, int ldx, T* out, int I, size_t count, int gated, int act) {
     pdl_enter();
     const size_t idx = blockIdx.x * (size_t)blockDim.x + threadIdx.x;
     if (idx >= count) return;
     const size_t r = idx / I;
     const int i = (int)(idx % I);
-    const float z = activation(x[r * ldx + i], act);
-    out[idx] = from_f32<T>(gated ? z * x[r * ldx + I + i] : z);
+    auto at = [&](size_t j) {
+        float v = x[j];
+        for (int s = 1; s < slices; ++s) v += x[s * slice_stride + j];
+        return v;
+    };
+    const float z = activation(at(r * ldx + i), act);
+    out[idx] = from_f32<T>(gated ? z * at(r * ldx + I + i) : z);
 }
 
 // One warp per token: scores s = sigmoid(logits), the k largest of s + bias (ties to the lower index), weights
-// s / (sum of the chosen s + 1e-20) * scale, or s * scale when renorm is 0.  logits: [slices, T, E], summed in order.
+// s / (sum of the chosen s + 1e-20) * scale, or s * scale when renorm is 0; squared at the end when `power` is 2.  logits: [slices, T, E], summed in order.
 // groups > 1: the experts form `groups` equal groups of neighbours; a group's worth is the sum of its two largest choice
 // values (its one value, if it has one expert), and only experts of the `keep` groups of most worth (ties to the lower
 // index) can be chosen.  Shared memory: E floats a warp (the choice values), E more (the scores) and `groups` more.
 __global__ void route_biased_kernel(const float* logits, int slices, size_t slice_stride, const float* bias, float scale, int T_, int E, int k,
-                                    int* sel_e, float* sel_w, int renorm, int groups, int keep) {
+                                    int* sel_e, float* sel_w, int renorm, int groups, int keep, int power) {
     pdl_enter();
     extern __shared__ float sc[];
     const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, warps = blockDim.x >> 5;
@@ -231,7 +237,10 @@ __global__ void route_biased_kernel(const float* logits, int slices, size_t slic
     const int last = lane < k ? ((k - 1 - lane) >> 5) * 32 + lane : -1;
     if (last >= 0) sel_w[(size_t)t * k + last] = mine, sel_e[(size_t)t * k + last] = mine_e;
     __syncwarp();
-    for (int j = lane; j < k; j += 32) sel_w[(size_t)t * k + j] = sel_w[(size_t)t * k + j] / den * scale;
+    for (int j = lane; j < k; j += 32) {
+        const float v = sel_w[(size_t)t * k + j] / den * scale;
+        sel_w[(size_t)t * k + j] = power == 2 ? v * v : v;
+    }
 }
 
 }  // namespace
@@ -257,23 +266,24 @@ Q6K_API int q6k_scaled_add_norm(float* h, const float* a, int a_slices, const fl
     return q6k_check_launch("scaled_add_norm");
 }
 
-Q6K_API int q6k_activate(const float* x, int ldx, void* out, int rows, int I, int gated, int act, int dtype, cudaStream_t st) {
+Q6K_API int q6k_activate(const float* x, int slices, long long slice_stride, int ldx, void* out, int rows, int I, int gated, int act, int dtype, cudaStream_t st) {
     if (rows == 0) return 0;
-    Q6K_REQUIRE(rows > 0 && I > 0 && ldx >= (gated ? 2 * I : I) && act >= 0 && act <= 2, "activate: bad sizes rows=%d I=%d ldx=%d act=%d", rows, I, ldx, act);
+    Q6K_REQUIRE(rows > 0 && I > 0 && ldx >= (gated ? 2 * I : I) && act >= 0 && act <= 3 && slices >= 1, "activate: bad sizes rows=%d I=%d ldx=%d act=%d", rows, I, ldx, act);
     const size_t count = (size_t)rows * I;
-    Q6K_DISPATCH(dtype, q6k_launch(activate_kernel<T>, (unsigned)((count + 255) / 256), 256, 0, st, x, ldx, (T*)out, I, count, gated, act););
+    Q6K_DISPATCH(dtype, q6k_launch(activate_kernel<T>, (unsigned)((count + 255) / 256), 256, 0, st, x, slices, (size_t)slice_stride, ldx, (T*)out, I, count, gated, act););
     return q6k_check_launch("activate");
 }
 
 Q6K_API int q6k_route_biased(const float* logits, int slices, const float* bias, float scale, int T_, int E, int k, int* sel_e, float* sel_w,
-                             int renorm, int groups, int keep, cudaStream_t st) {
+                             int renorm, int groups, int keep, int power, cudaStream_t st) {
     if (T_ == 0) return 0;
     Q6K_REQUIRE(T_ > 0 && E > 0 && k > 0 && k <= E && slices >= 1, "route_biased: bad sizes T=%d E=%d k=%d slices=%d", T_, E, k, slices);
     Q6K_REQUIRE(E <= 4096, "route_biased: %d experts exceed the supported 4096", E);
     Q6K_REQUIRE(groups >= 1 && E % groups == 0 && keep >= 1 && keep <= groups && k <= keep * (E / groups),
                 "route_biased: %d experts in %d groups, %d kept, %d chosen", E, groups, keep, k);
+    Q6K_REQUIRE(power == 1 || power == 2, "route_biased: weights to the power %d", power);
     const int warps = E <= 1024 ? 4 : 1;
     q6k_launch(route_biased_kernel, (T_ + warps - 1) / warps, warps * 32, (size_t)warps * (2 * E + groups) * sizeof(float), st, logits, slices,
-               (size_t)T_ * E, bias, scale, T_, E, k, sel_e, sel_w, renorm, groups, keep);
+               (size_t)T_ * E, bias, scale, T_, E, k, sel_e, sel_w, renorm, groups, keep, power);
     return q6k_check_launch("route_biased");
 }

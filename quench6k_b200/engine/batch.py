@@ -50,6 +50,8 @@ class StepContext:
     leave_bias: bool = False                      # a block that adds a per-column bias with the sublayer's result sets it: a mixer whose
                                                   # last projection has a bias then hands the bias over in `left_bias` instead of adding it
     left_bias: Optional[torch.Tensor] = None
+    takes_pair: bool = False                      # a block whose add can norm two results side by side sets it: a mixer may then return a
+                                                  # parts.base.NormedPair instead of making the sum itself
     position: int = 0                             # the executed position (index into the model's order) whose block is running
     side_rows: Optional[torch.Tensor] = None      # FP32 [T, columns]: the tokens' rows of the model's side table, if it has one
 

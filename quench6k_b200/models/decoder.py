@@ -13,7 +13,7 @@ import torch
 
 from .. import ops
 from ..parts import linear
-from ..parts.base import (BLOCKS, EMBED_ADDS, FEED_FORWARDS, MIXERS, NORMS, CacheRequest, LayerCache, Runtime, WeightedRows, make_part,
+from ..parts.base import (BLOCKS, CONNECTIONS, EMBED_ADDS, FEED_FORWARDS, MIXERS, NORMS, CacheRequest, LayerCache, Runtime, Streams, WeightedRows, make_part,
                           to_operand)
 from ..spec import ModelSpec, TensorSpec
 
@@ -37,6 +37,12 @@ class DecoderModel:
                     after["norm2b"] = make_part(NORMS, "norm", ls.post_norm, size=D)
             if ls.side is not None:
                 after["side"] = make_part(FEED_FORWARDS, "feed-forward", ls.side, hidden_size=D)
+            if ls.connection is not None:
+                after["connect1"] = make_part(CONNECTIONS, "connection", ls.connection)
+                if ffn is not None:
+                    after["connect2"] = make_part(CONNECTIONS, "connection", ls.connection)
+            if (ls.connection is not None) != (spec.streams > 0):
+                raise ValueError(f"layer {ls.prefix!r}: a residual of several streams and its connections go together")
             self.blocks.append(BLOCKS[ls.block](norm1, mixer, norm2, ffn, **after, **ls.block_params))
         self.embed_norm = make_part(NORMS, "norm", spec.embed_norm, size=D) if spec.embed_norm is not None else None
         self.embed_add = make_part(EMBED_ADDS, "embedding add", spec.embed_add, hidden_size=D) if spec.embed_add is not None else None
@@ -48,6 +54,8 @@ class DecoderModel:
         self.readd = set(spec.readd_embedding)
         if any(not 0 < p < len(self.order) for p in self.readd):
             raise ValueError("readd_embedding names a position outside 1..executed layers - 1")
+        if spec.streams and self.readd:
+            raise ValueError("the embedding output is not added again to a residual of several streams")
         self.rt: Optional[Runtime] = None
 
     # ------------------------------------------------------------------ declaration
@@ -102,6 +110,7 @@ class DecoderModel:
                 pre = ls.prefix + s.sub_names[sub]
                 part.bind(lambda n, pre=pre: get(pre + n), rt)
         self.final_norm.bind(lambda n: get(s.final_norm_prefix + n), rt)
+        self.stream_sum = torch.ones(s.streams, dtype=torch.float32, device=rt.device) if s.streams else None
         self.head = self.embed if s.head_name is None else to_operand(get(s.head_name), rt)
 
     # ------------------------------------------------------------------ one step
@@ -119,6 +128,8 @@ class DecoderModel:
         if self.side_table is not None:
             ops.current_tag = "embedding.side"
             ctx.side_rows = ops.embed(ctx.token_ids, self.side_table, fed=ctx.fed)
+        if self.spec.streams:
+            h = Streams(h, self.spec.streams)
         h0 = h.clone() if self.readd else None      # the embedding output, for the passes of a repeated span that take it again
         pending = None                      # an add into h that a block has left to the next norm
         for p, i in enumerate(self.order):
@@ -135,6 +146,11 @@ class DecoderModel:
             pending = block.forward(h, ctx, caches[p], states[p], pending)
         if ctx.n_logit_rows == 0:
             return None
+        if self.spec.streams:               # the last add, the sum of the streams and the last norm: one pass over the wanted rows
+            ops.current_tag = "norm.final"
+            xn = h.step(pending, self.stream_sum, self.final_norm, rows=ctx.logit_rows)
+            ops.current_tag = "lm_head"
+            return linear.matmul(xn, self.head, self.rt)
         # an add that is left: the last norm makes it if it can (it normalises picked rows only, so a sublayer result that
         # passes a norm of its own is added first, for all rows)
         if pending is not None and not (isinstance(pending, WeightedRows) and self.final_norm.fuses_weighted_rows):

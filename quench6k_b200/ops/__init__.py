@@ -57,7 +57,7 @@ def _need(t: torch.Tensor, name: str, dtype=None, shape=None):
 
 
 # kernels launched per exported function (for launch accounting in benchmarks)
-_LAUNCHES = {"q6k_gated_delta": 1, "q6k_attention_flex_mma": 2, "q6k_selective_scan": 1, "q6k_moe_permute": 3, "q6k_moe_plan": 3, "q6k_gemm_tc": 1, "q6k_attention_mma": 2, "q6k_argmax": 2, "q6k_gemm_tc_pairs_scratch": 0}
+_LAUNCHES = {"q6k_gated_delta": 1, "q6k_delta_channel": 1, "q6k_attention_flex_mma": 2, "q6k_selective_scan": 1, "q6k_moe_permute": 3, "q6k_moe_plan": 3, "q6k_gemm_tc": 1, "q6k_attention_mma": 2, "q6k_argmax": 2, "q6k_gemm_tc_pairs_scratch": 0}
 launch_count = 0
 
 
@@ -563,10 +563,11 @@ def gemm_skinny(x: torch.Tensor, w: torch.Tensor, w2: Optional[torch.Tensor] = N
 def qk_prep(qkv: torch.Tensor, Hq: int, Hkv: int, hd: int, q_norm, k_norm, eps: float, rotary,
             positions: torch.Tensor, req_of_token: torch.Tensor, block_table: Optional[torch.Tensor], page_size: int,
             k_pages: Optional[torch.Tensor], v_pages: Optional[torch.Tensor], out_dtype: torch.dtype, bias: Optional[torch.Tensor] = None,
-            values_are_keys: bool = False) -> torch.Tensor:
+            values_are_keys: bool = False, value_norm: bool = False) -> torch.Tensor:
     """QK-norm, rotation, q -> out_dtype [T, Hq, hd]; k, v -> their pages (when k_pages is given).
     bias: FP32, one entry per column of a row (q, k, v side by side), added to the summed product first.  values_are_keys:
     the rows hold q and k only, and a key's value is the key as projected (bias included, before norm and rotation).
+    value_norm: a head's value is divided by its root mean square (eps, no weight) before it is stored.
     rotary: None, or (inv_freq float32 [rotary_dim / 2] on the device, rotary_dim, neighbours): the
     first rotary_dim dimensions of every q and k head turn by position * inv_freq[pair], paired by
     halves (d with d + rotary_dim / 2) or, neighbours=True, 2i with 2i + 1.
@@ -605,7 +606,7 @@ def qk_prep(qkv: torch.Tensor, Hq: int, Hkv: int, hd: int, q_norm, k_norm, eps: 
     _call("q6k_qk_prep", _ptr(qkv), _i(qkv.stride(0)), _i(splits), _ll(split_stride), _i(T), _i(Hq), _i(Hkv), _i(hd), _ptr(q_norm), _ptr(k_norm), _f(eps),
           _ptr(inv_freq), _i(rotary_dim), _i(1 if neighbours else 0), _ptr(positions), _ptr(req_of_token), _ptr(block_table),
           _i(max_blocks), _i(page_size), _i(k_pages.shape[1] if write else 0), _ptr(q), _ptr(k_pages), _ptr(v_pages),
-          _i(1 if write else 0), _i(dtype_code(out_dtype)), _ptr(bias), _i(1 if values_are_keys else 0), _stream())
+          _i(1 if write else 0), _i(dtype_code(out_dtype)), _ptr(bias), _i(1 if values_are_keys else 0), _i(1 if value_norm else 0), _stream())
     return q
 
 
@@ -1146,11 +1147,12 @@ def selective_scan_segments(q_lens, device):
 def qkv_pages(qkv: torch.Tensor, Hq: int, Hkv: int, hd: int, vd: int, q_norm, k_norm, eps: float, rotary, positions: torch.Tensor,
               req_of_token: torch.Tensor, block_table: Optional[torch.Tensor], page_size: int, k_pages: Optional[torch.Tensor],
               v_pages: Optional[torch.Tensor], out_dtype: torch.dtype, v_heads: Optional[int] = None, bias: Optional[torch.Tensor] = None,
-              values_are_keys: bool = False) -> torch.Tensor:
+              values_are_keys: bool = False, value_norm: bool = False) -> torch.Tensor:
     """qk_prep for keys and values of different widths: qkv FP32 [T, Hq hd + Hkv hd + Hv vd] (or split-K slices of it);
     q -> [T, Hq, hd]; k -> pages [Hkv, P, page, hd]; v -> pages [Hv, P, page, vd].  v_heads: Hv, if it is not Hkv.
     bias: FP32, one entry per column of a row, added to the summed product first.  values_are_keys: the rows hold q and k
-    only, and a key's value is the key as projected (bias included, before norm and rotation)."""
+    only, and a key's value is the key as projected (bias included, before norm and rotation).  value_norm: a head's value is
+    divided by its root mean square (eps, no weight) before it is stored."""
     Hv = v_heads or Hkv
     v_cols = 0 if values_are_keys else Hv * vd
     if bias is not None:
@@ -1177,27 +1179,30 @@ def qkv_pages(qkv: torch.Tensor, Hq: int, Hkv: int, hd: int, vd: int, q_norm, k_
           _ptr(k_norm), _f(eps), _ptr(inv_freq), _i(rotary_dim), _i(1 if neighbours else 0), _ptr(positions), _ptr(req_of_token),
           _ptr(block_table), _i(block_table.shape[1] if block_table is not None else 1), _i(page_size),
           _i(k_pages.shape[1] if write else 0), _ptr(q), _ptr(k_pages), _ptr(v_pages), _i(1 if write else 0),
-          _i(dtype_code(out_dtype)), _i(Hv), _ptr(bias), _i(1 if values_are_keys else 0), _stream())
+          _i(dtype_code(out_dtype)), _i(Hv), _ptr(bias), _i(1 if values_are_keys else 0), _i(1 if value_norm else 0), _stream())
     return q
 
 
 def latent_prep(x: torch.Tensor, H: int, dim: int, rd: int, rank: int, c_weight: Optional[torch.Tensor], eps: float,
                 inv_freq: Optional[torch.Tensor], turn: int, positions: torch.Tensor, req_of_token: torch.Tensor, block_table: torch.Tensor,
-                page_size: int, pages: torch.Tensor, neighbours: bool = False, write: bool = True):
+                page_size: int, pages: torch.Tensor, neighbours: bool = False, write: bool = True, latent=None):
     """x FP32 [T, H (dim + rd) + rank + rd] -> (qn [H, T, dim], qr [H, T, rd]) in the pages' dtype, and the token's row
     [RMS-normed latent | rotated shared key part] into pages [1, P, page, rank + rd].  neighbours: the rotation pairs
     dimension 2i with 2i+1 instead of i with i + turn/2.  write=False: a layer that reads another layer's pages; x then
-    holds the queries only and nothing is written."""
+    holds the queries only and nothing is written.  latent = (rows FP32 [T, *], column): the latent and the shared key part
+    are read there; x then holds the queries only."""
     _need(x, "x", torch.float32)
     T = x.shape[0]
-    if x.shape[1] < H * (dim + rd) + (rank + rd if write else 0) or tuple(pages.shape[2:]) != (page_size, rank + rd) or pages.shape[0] != 1:
+    xc, col = latent if latent is not None else (x, H * (dim + rd))
+    _need(xc, "latent rows", torch.float32)
+    if x.shape[1] < H * (dim + rd) or (write and (xc.shape[0] != T or xc.shape[1] < col + rank + rd)) or tuple(pages.shape[2:]) != (page_size, rank + rd) or pages.shape[0] != 1:
         raise KernelError("latent_prep: shapes disagree")
     _need(pages, "pages")
     if write:
         _need(c_weight, "c_weight", torch.float32, (rank,))
     qn = torch.empty((H, T, dim), dtype=pages.dtype, device=x.device)
     qr = torch.empty((H, T, rd), dtype=pages.dtype, device=x.device)
-    _call("q6k_latent_prep", _ptr(x), _i(x.stride(0)), _i(T), _i(H), _i(dim), _i(rd), _i(rank), _ptr(c_weight if write else None), _f(eps),
+    _call("q6k_latent_prep", _ptr(x), _i(x.stride(0)), ctypes.c_void_p(xc.data_ptr() + 4 * col if write else 0), _i(xc.stride(0)), _i(T), _i(H), _i(dim), _i(rd), _i(rank), _ptr(c_weight if write else None), _f(eps),
           _ptr(inv_freq), _i(turn), _i(1 if neighbours else 0), _ptr(positions), _ptr(req_of_token), _ptr(block_table), _i(block_table.shape[1]),
           _i(page_size), _ptr(qn), _ptr(qr), _ptr(pages if write else None), _i(dtype_code(pages.dtype)), _stream())
     return qn, qr
@@ -1389,18 +1394,19 @@ OUT_GATES = {"silu": 0, "sigmoid": 1}
 def delta_out(o: torch.Tensor, p: torch.Tensor, g_col: int, w: torch.Tensor, eps: float, H: int, dv: int, out_dtype: torch.dtype,
               gate: str = "silu") -> torch.Tensor:
     """out_dtype(o / rms(o) * w * gate(g)) per (row, head): o FP32 [T, H dv], g in p's columns from g_col on; gate: silu or
-    sigmoid.  With H = 1 and dv the width of all heads together, the heads are normed as one vector."""
+    sigmoid.  w: FP32 [dv], shared by the heads, or [H, dv].  With H = 1 and dv the width of all heads together, the heads are
+    normed as one vector."""
     if gate not in OUT_GATES:
         raise KernelError(f"delta_out: unknown gate {gate!r}; known: {', '.join(OUT_GATES)}")
     _need(o, "o", torch.float32)
     _need(p, "p", torch.float32)
-    _need(w, "w", torch.float32, (dv,))
+    _need(w, "w", torch.float32, (dv,) if w.dim() == 1 else (H, dv))
     T = o.shape[0]
     if o.shape[1] != H * dv or p.shape[0] != T or g_col + H * dv > p.shape[1]:
         raise KernelError("delta_out: shapes disagree")
     out = torch.empty((T, H * dv), dtype=out_dtype, device=o.device)
     _call("q6k_delta_out", _ptr(o), _ptr(p), _i(p.stride(0)), _i(g_col), _ptr(w), _f(eps), _ptr(out), _i(T), _i(H), _i(dv), _i(dtype_code(out_dtype)),
-          _i(OUT_GATES[gate]), _stream())
+          _i(OUT_GATES[gate]), _i(dv if w.dim() == 2 else 0), _stream())
     return out
 
 
@@ -1452,22 +1458,24 @@ def scaled_add_norm(h: torch.Tensor, a: Optional[torch.Tensor], b: Optional[torc
 
 
 def activate(x: torch.Tensor, I: int, gated: bool, act: str, out_dtype: torch.dtype) -> torch.Tensor:
-    """out_dtype(act(x[:, :I]) * x[:, I:2 I]) when gated, else out_dtype(act(x[:, :I])); x FP32."""
+    """out_dtype(act(x[:, :I]) * x[:, I:2 I]) when gated, else out_dtype(act(x[:, :I])); x FP32 [T, N], or [slices, T, N]
+    partial sums (added in order).  act: one of ACTIVATIONS, or "tanh"."""
     _need(x, "x", torch.float32)
-    if act not in ACTIVATIONS:
+    slices, stride, T, N = _slices_of(x)
+    if act not in ACTIVATIONS and act != "tanh":
         raise KernelError(f"activate: unknown activation {act!r}")
-    out = torch.empty((x.shape[0], I), dtype=out_dtype, device=x.device)
-    _call("q6k_activate", _ptr(x), _i(x.stride(0)), _ptr(out), _i(x.shape[0]), _i(I), _i(1 if gated else 0), _i(ACTIVATIONS[act]),
+    out = torch.empty((T, I), dtype=out_dtype, device=x.device)
+    _call("q6k_activate", _ptr(x), _i(slices), _ll(stride), _i(N), _ptr(out), _i(T), _i(I), _i(1 if gated else 0), _i(3 if act == "tanh" else ACTIVATIONS[act]),
           _i(dtype_code(out_dtype)), _stream())
     return out
 
 
-def route_biased(logits: torch.Tensor, k: int, bias: Optional[torch.Tensor], scale: float, renorm: bool = True, groups=None):
+def route_biased(logits: torch.Tensor, k: int, bias: Optional[torch.Tensor], scale: float, renorm: bool = True, groups=None, power: int = 1):
     """(sel_e int32 [T, k], sel_w float32 [T, k]): per row the k experts with the largest sigmoid(logit) + bias (ties to the
     lower index); weights sigmoid(logit) / (their sum + 1e-20) * scale, or sigmoid(logit) * scale without renorm.
     groups = (count, keep): the experts form `count` equal groups of neighbours, a group's worth is the sum of its two
     largest choice values, and only experts of the `keep` groups of most worth can be chosen.
-    logits: [T, E] or [slices, T, E] partial sums."""
+    power = 2: the weights leave squared.  logits: [T, E] or [slices, T, E] partial sums."""
     count, keep = groups if groups is not None else (1, 1)
     _need(logits, "logits", torch.float32)
     slices = logits.shape[0] if logits.dim() == 3 else 1
@@ -1477,7 +1485,7 @@ def route_biased(logits: torch.Tensor, k: int, bias: Optional[torch.Tensor], sca
     sel_e = torch.empty((T, k), dtype=torch.int32, device=logits.device)
     sel_w = torch.empty((T, k), dtype=torch.float32, device=logits.device)
     _call("q6k_route_biased", _ptr(logits), _i(slices), _ptr(bias), _f(scale), _i(T), _i(E), _i(k), _ptr(sel_e), _ptr(sel_w),
-          _i(1 if renorm else 0), _i(count), _i(keep), _stream())
+          _i(1 if renorm else 0), _i(count), _i(keep), _i(power), _stream())
     return sel_e, sel_w
 
 
@@ -1564,3 +1572,195 @@ def retention(p: torch.Tensor, q_col: int, k_col: int, v_col: int, decay: torch.
     _call("q6k_retention", _ptr(p), _i(p.stride(0)), _i(q_col), _i(k_col), _i(v_col), _ptr(decay), _ptr(state), _ptr(q_start), _ptr(slot_ids),
           _i(R), _ptr(o), _i(H), _i(dk), _i(dv), _stream())
     return o
+
+
+def token_shift(x: torch.Tensor, mu: torch.Tensor, prev: torch.Tensor, req_of_token: torch.Tensor, q_start: torch.Tensor,
+                slot_ids: torch.Tensor) -> torch.Tensor:
+    """out[j, t] = x + (x' - x) mu[j] in x's dtype, x' the row before t in its request: the n mixes of every token with the one
+    before it, [n, T, D].  x: [T, D]; mu: FP32 [n, D]; prev: FP32 [slots, D], the last row of the request's earlier portions
+    (zeros at its start), moved on to this portion's last row."""
+    _need(x, "x")
+    T, D = x.shape
+    n = mu.shape[0]
+    _need(mu, "mu", torch.float32, (n, D))
+    _need(prev, "prev", torch.float32)
+    if prev.shape[-1] != D:
+        raise KernelError("token_shift: the state does not match the rows")
+    out = torch.empty((n, T, D), dtype=x.dtype, device=x.device)
+    _call("q6k_token_shift", _ptr(x), _ptr(mu), _i(n), _ptr(prev), _ptr(req_of_token), _ptr(q_start), _ptr(slot_ids), _ptr(out), _i(T), _i(D),
+          _i(dtype_code(x.dtype)), _stream())
+    return out
+
+
+def time_mix(r: torch.Tensor, k: torch.Tensor, v: torch.Tensor, w: torch.Tensor, w0: torch.Tensor, u: torch.Tensor, state: torch.Tensor,
+             q_start: torch.Tensor, slot_ids: torch.Tensor, R: int) -> torch.Tensor:
+    """Per request and head, in token order: o = S^T r + (sum_x u[x] k[x] r[x]) v, then S <- diag(exp(-exp(w + w0))) S + k v^T.
+    r, k: FP32 [T, H dk]; v: FP32 [T, H dv]; w: FP32 [T, H dk], overwritten by the decays; w0, u: FP32 [H, dk]; state FP32
+    [slots, H, dk, dv], updated in place.  Returns FP32 o [T, H dv]."""
+    for nm, t in (("r", r), ("k", k), ("v", v), ("w", w), ("w0", w0), ("u", u), ("state", state)):
+        _need(t, nm, torch.float32)
+    H, dk = u.shape
+    dv = state.shape[-1]
+    T = r.shape[0]
+    if (tuple(state.shape[1:]) != (H, dk, dv) or tuple(r.shape) != (T, H * dk) or k.shape != r.shape or w.shape != r.shape or w0.numel() != H * dk
+            or tuple(v.shape) != (T, H * dv) or dv != dk):
+        raise KernelError("time_mix: shapes disagree")
+    bonus = torch.empty((T, H), dtype=torch.float32, device=r.device)
+    _call("q6k_time_mix_prep", _ptr(r), _ptr(k), _i(H * dk), _ptr(w), _ptr(w0), _ptr(u), _ptr(bonus), _i(T), _i(H), _i(dk), _stream())
+    o = torch.empty((T, H * dv), dtype=torch.float32, device=r.device)
+    _call("q6k_time_mix", _ptr(r), _ptr(k), _ptr(v), _i(H * dk), _ptr(w), _ptr(bonus), _ptr(state), _ptr(q_start), _ptr(slot_ids), _i(R), _ptr(o), _i(H),
+          _i(dk), _i(dv), _stream())
+    return o
+
+
+# --------------------------------------------------------------------------- a delta rule with a decay per key channel
+@functools.lru_cache(maxsize=None)
+def delta_channel_max_dim() -> int:
+    lib = library()
+    lib.q6k_delta_channel_max_dim.restype = ctypes.c_int
+    return lib.q6k_delta_channel_max_dim()
+
+
+@functools.lru_cache(maxsize=None)
+def _delta_channel_scratch(H: int, dk: int) -> int:
+    lib = library()
+    lib.q6k_delta_channel_scratch.restype = ctypes.c_longlong
+    return lib.q6k_delta_channel_scratch(_i(H), _i(dk))
+
+
+def delta_channel(u: torch.Tensor, p: torch.Tensor, b_col: int, a: torch.Tensor, a_col: int, A_log: torch.Tensor, dt_bias: torch.Tensor,
+                  state: torch.Tensor, req_of_token: torch.Tensor, q_start: torch.Tensor, slot_ids: torch.Tensor, R: int, H: int, G: int, dk: int,
+                  dv: int, prepare: bool = False) -> torch.Tensor:
+    """gated_delta with one decay per head and key channel: S <- diag(g) S; u = beta (v - S^T k); S <- S + k u^T; o = S^T q with
+    g = exp(-exp(A_log[h]) softplus(a + dt_bias)).  a: FP32 [T, *] with the H dk decay inputs from a_col on, dt_bias: FP32
+    [H dk]; the rest as in gated_delta.  prepare: a kernel of its own makes what does not depend on the state (steps with long
+    portions); else the recurrence makes it itself.  The results are the same bit for bit."""
+    _need(u, "u", torch.float32)
+    _need(p, "p", torch.float32)
+    _need(a, "a", torch.float32)
+    _need(A_log, "A_log", torch.float32, (H,))
+    _need(dt_bias, "dt_bias", torch.float32, (H * dk,))
+    _need(state, "state", torch.float32)
+    T = u.shape[0]
+    if (tuple(state.shape[1:]) != (H, dv, dk) or u.shape[1] < 2 * G * dk + H * dv or p.shape[0] != T or b_col + H > p.shape[1] or a.shape[0] != T
+            or a_col + H * dk > a.shape[1]):
+        raise KernelError("delta_channel: shapes disagree")
+    o = torch.empty((T, H * dv), dtype=torch.float32, device=u.device)
+    scratch = torch.empty(T * _delta_channel_scratch(H, dk), dtype=torch.float32, device=u.device) if prepare else None
+    _call("q6k_delta_channel", _ptr(u), _i(u.stride(0)), _ptr(p), _i(p.stride(0)), _i(b_col), _ptr(a), _i(a.stride(0)), _i(a_col), _ptr(A_log), _ptr(dt_bias),
+          _ptr(scratch), _ptr(state), _ptr(req_of_token), _ptr(q_start), _ptr(slot_ids), _ptr(o), _i(T), _i(R), _i(H), _i(G), _i(dk), _i(dv), _stream())
+    return o
+
+
+# --------------------------------------------------------------------------- heads' gates, norms of some columns
+def gate_heads(a: torch.Tensor, H: int, p: torch.Tensor, col: int) -> None:
+    """a[t, h] *= sigmoid(p[t, col + h]) in place: a [T, H n] in either dtype, p FP32 [T, *] or [slices, T, *] partial sums."""
+    _need(a, "a")
+    _need(p, "p", torch.float32)
+    slices, stride, T, N = _slices_of(p)
+    if a.shape[0] != T or a.shape[1] % H or col + H > N:
+        raise KernelError("gate_heads: shapes disagree")
+    _call("q6k_gate_heads", _ptr(a), _ptr(p), _i(slices), _ll(stride), _i(N), _i(col), _i(T), _i(H), _i(a.shape[1] // H), _i(dtype_code(a.dtype)), _stream())
+
+
+def norm_columns(x: torch.Tensor, col: int, n: int, w: torch.Tensor, eps: float, out_dtype: torch.dtype) -> torch.Tensor:
+    """out_dtype(c * rsqrt(mean(c^2) + eps) * w) for the columns c = x[t, col : col + n] of FP32 rows."""
+    _need(x, "x", torch.float32)
+    _need(w, "w", torch.float32, (n,))
+    if col + n > x.shape[1]:
+        raise KernelError("norm_columns: shapes disagree")
+    out = torch.empty((x.shape[0], n), dtype=out_dtype, device=x.device)
+    _call("q6k_norm_columns", _ptr(x), _i(x.stride(0)), _i(col), _i(n), _ptr(w), _f(eps), _ptr(out), _i(x.shape[0]), _i(dtype_code(out_dtype)), _stream())
+    return out
+
+
+# --------------------------------------------------------------------------- a residual of several streams
+@functools.lru_cache(maxsize=None)
+def hyper_max_streams() -> int:
+    lib = library()
+    lib.q6k_hyper_max_streams.restype = ctypes.c_int
+    return lib.q6k_hyper_max_streams()
+
+
+def normed_pair(a: torch.Tensor, bias: Optional[torch.Tensor], b: torch.Tensor, wa: torch.Tensor, wb: torch.Tensor, mult: float, eps: float) -> torch.Tensor:
+    """FP32 mult * (norm(a + bias) wa + norm(b) wb), each over its root mean square along the row; a, b FP32 [T, D] or
+    [slices, T, D] partial sums, bias FP32 [D] or None."""
+    _need(a, "a", torch.float32)
+    _need(b, "b", torch.float32)
+    na, sa, T, D = _slices_of(a)
+    nb, sb, T2, D2 = _slices_of(b)
+    if (T, D) != (T2, D2):
+        raise KernelError("normed_pair: shapes disagree")
+    for nm, t in (("bias", bias), ("wa", wa), ("wb", wb)):
+        if t is not None:
+            _need(t, nm, torch.float32, (D,))
+    out = torch.empty((T, D), dtype=torch.float32, device=a.device)
+    _call("q6k_normed_pair", _ptr(a), _i(na), _ptr(bias), _ptr(b), _i(nb), _ll(T * D), _ptr(wa), _ptr(wb), _f(mult), _f(eps), _ptr(out), _i(T), _i(D), _stream())
+    return out
+
+
+def hyper_step(x: torch.Tensor, S: int, add=None, read=None, rows: Optional[torch.Tensor] = None, out_dtype: torch.dtype = torch.float32):
+    """One pass over a residual of S streams.  x: FP32 [T, S, D], or [T, D] while all streams are equal.
+    add = {"a", "bias", "weighted", "pair", "mix", "out"}: x_t <- sum_s mix[s, t] x_s + out[t] y for all streams at once, y = a (FP32
+    [T, D] or [slices, T, D] partial sums) + bias (FP32 [D]) + weighted rows (as in `combine`), each optional; or, with pair = (b, wa, wb,
+    mult, eps), y = mult (norm(a + bias) wa + norm(b) wb).  mix: FP32 [S, S] (from, to); out: FP32 [S].
+    read = (weights FP32 [S], norm weight FP32 [D], eps): the norm of sum_t weights[t] x_t in out_dtype.
+    rows: read these rows only, and store no streams.  Returns (streams [T, S, D] as they then stand, or x itself when nothing was
+    added or rows are picked; the norm or None)."""
+    _need(x, "x", torch.float32)
+    broadcast = x.dim() == 2
+    T, D = x.shape[0], x.shape[-1]
+    if not broadcast and x.shape[1] != S:
+        raise KernelError(f"hyper_step: {x.shape[1]} streams, expected {S}")
+    a = bias = py = pair_row = pw = b = wa = wb = mix = out_w = None
+    na = nb = 1
+    K, mult, eps = 0, 1.0, read[2] if read is not None else 0.0
+    if add is not None:
+        a, bias, mix, out_w = add.get("a"), add.get("bias"), add["mix"], add["out"]
+        _need(mix, "mix", torch.float32, (S, S))
+        _need(out_w, "out", torch.float32, (S,))
+        if bias is not None:
+            _need(bias, "bias", torch.float32, (D,))
+        if a is not None:
+            _need(a, "a", torch.float32)
+            na, _, ta, da = _slices_of(a)
+            if (ta, da) != (T, D):
+                raise KernelError("hyper_step: the sublayer's result does not match the streams")
+        if add.get("weighted") is not None:
+            py, pair_row, pw = add["weighted"]
+            _need(py, "weighted rows", torch.float32)
+            _need(pw, "weights", torch.float32)
+            K = pw.shape[1]
+            if pair_row is not None:
+                _need(pair_row, "pair_row", torch.int32)
+            if pw.shape[0] != T or py.shape[1] != D or py.shape[0] < T * K or (pair_row is not None and pair_row.numel() != T * K):
+                raise KernelError("hyper_step: the weighted rows do not match the streams")
+        if add.get("pair") is not None:
+            b, wa, wb, mult, pair_eps = add["pair"]
+            _need(b, "b", torch.float32)
+            nb, _, tb, db = _slices_of(b)
+            _need(wa, "wa", torch.float32, (D,))
+            _need(wb, "wb", torch.float32, (D,))
+            if a is None or (tb, db) != (T, D) or py is not None:
+                raise KernelError("hyper_step: two normed results of one shape, without routed rows")
+            if read is not None and pair_eps != eps:
+                raise KernelError("hyper_step: the results' norms and the sublayer's share one eps")
+            eps = pair_eps
+        if a is None and py is None and bias is None:
+            raise KernelError("hyper_step: nothing to add")
+    in_w = norm_w = out = None
+    R = T if rows is None else rows.numel()
+    if read is not None:
+        in_w, norm_w = read[0], read[1]
+        _need(in_w, "stream weights", torch.float32, (S,))
+        _need(norm_w, "norm weight", torch.float32, (D,))
+        out = torch.empty((R, D), dtype=out_dtype, device=x.device)
+    if rows is not None:
+        _need(rows, "rows", torch.int32)
+    dst = x if add is None or rows is not None else torch.empty((T, S, D), dtype=torch.float32, device=x.device) if broadcast else x
+    if add is None and read is None:
+        return x, None
+    _call("q6k_hyper_step", _ptr(x), _i(1 if broadcast else 0), _ptr(dst if add is not None and rows is None else None), _ptr(a), _i(na), _ll(T * D), _ptr(bias),
+          _ptr(py), _ptr(pair_row), _ptr(pw), _i(K), _ptr(b), _i(nb), _ptr(wa), _ptr(wb), _f(mult), _ptr(mix), _ptr(out_w), _ptr(in_w), _ptr(norm_w), _f(eps),
+          _ptr(out), _ptr(rows), _i(R), _i(S), _i(D), _i(dtype_code(out_dtype)), _stream())
+    return dst, out

@@ -19,7 +19,9 @@ value); a cap on the scaled scores
 (`softcap`: s -> c tanh(s / c)); and difference attention (`maps=2` with `diff`): every head attends twice, with queries
 and keys of its own per map (q and k hold a head's maps side by side, the q/k norm weights are shared by all heads and
 maps) over the same values, and the head's result is o = a1 - L a2 divided by its root mean square over the value
-width, times (1 - diff), where L = exp(lq1 . lk1) - exp(lq2 . lk2) + diff is one number made from four stored vectors."""
+width, times (1 - diff), where L = exp(lq1 . lk1) - exp(lq2 . lk2) + diff is one number made from four stored vectors;
+values divided by their root mean square before they are cached (`value_norm`); and a gate per head on the head's result,
+sigmoid of one more projection of the input (`head_gate`, H more rows of the stacked product)."""
 from __future__ import annotations
 
 import math
@@ -42,7 +44,8 @@ class Attention(Mixer):
                  norm_init: str = "ones", sink_std: float = 1.0, v_dim: Optional[int] = None, scale: Optional[float] = None,
                  chunk: Optional[int] = None, talk: bool = False, names=None, bias: bool = False, conv: Optional[int] = None,
                  o_bias: bool = False, fixed_sink: Optional[float] = None, qk_norm_weight: bool = True, values_are_keys: bool = False,
-                 softcap: Optional[float] = None, maps: int = 1, diff: Optional[float] = None):
+                 softcap: Optional[float] = None, maps: int = 1, diff: Optional[float] = None, value_norm: bool = False,
+                 head_gate: bool = False):
         if num_heads % num_kv_heads:
             raise ValueError(f"{num_heads} query heads are not a multiple of {num_kv_heads} KV heads")
         self.D, self.Hq, self.Hkv, self.hd = hidden_size, num_heads, num_kv_heads, head_dim
@@ -58,6 +61,11 @@ class Attention(Mixer):
         self.diff = float(diff) if diff is not None else None
         if self.maps not in (1, 2) or (self.maps == 2) != (self.diff is not None):
             raise ValueError(f"{maps} maps with diff {diff!r}: difference attention has two maps and a diff, plain attention one and none")
+        self.value_norm, self.head_gate = bool(value_norm), bool(head_gate)
+        if self.maps > 1 and self.head_gate:
+            raise ValueError("a gate per head goes with one map")
+        if self.value_norm and self.pos.rotary_table() is None and not self.pos.is_identity:
+            raise ValueError("normed values take a rotation of pairs or no position encoding")
         if sinks and fixed_sink is not None:
             raise ValueError("learned sinks and a fixed sink exclude each other")
         if self.values_are_keys and (self.vd != head_dim or self.maps > 1 or conv):
@@ -81,10 +89,13 @@ class Attention(Mixer):
         self.names = {"q": "q_proj.weight", "k": "k_proj.weight", "v": "v_proj.weight", "o": "o_proj.weight", "q_norm": "q_norm.weight",
                       "k_norm": "k_norm.weight", "sinks": "sinks", "talk": "talk.weight", "q_bias": "q_proj.bias", "k_bias": "k_proj.bias",
                       "v_bias": "v_proj.bias", "q_conv": "q_conv.weight", "k_conv": "k_conv.weight", "v_conv": "v_conv.weight",
-                      "o_bias": "o_proj.bias", "lq1": "lambda_q1", "lk1": "lambda_k1", "lq2": "lambda_q2", "lk2": "lambda_k2", **(names or {})}
+                      "o_bias": "o_proj.bias", "lq1": "lambda_q1", "lk1": "lambda_k1", "lq2": "lambda_q2", "lk2": "lambda_k2", "gate": "g_proj.weight",
+                      **(names or {})}
         # rows of the stacked projection: a head's maps side by side in q and k, one value head per KV head
         self.nq, self.nk = num_heads * self.maps * head_dim, num_kv_heads * self.maps * head_dim
         self.nv = 0 if self.values_are_keys else num_kv_heads * self.vd
+        self.g_col = self.nq + self.nk + self.nv                          # the heads' gates come last, padded to a multiple of 8 rows
+        self.ng = -(-(self.g_col + num_heads) // 8) * 8 - self.g_col if self.head_gate else 0
 
     def tensors(self):
         D, Hq, Hkv, hd, n = self.D, self.Hq, self.Hkv, self.hd, self.names
@@ -92,6 +103,8 @@ class Attention(Mixer):
         if not self.values_are_keys:
             out.append(TensorSpec(n["v"], (self.nv, D)))
         out.append(TensorSpec(n["o"], (D, Hq * self.vd)))
+        if self.head_gate:
+            out.append(TensorSpec(n["gate"], (Hq, D)))
         if self.qk_norm and self.qk_norm_weight:
             init = ("ones",) if self.norm_init == "ones" else ("ones_plus", 0.1)
             out += [TensorSpec(n["q_norm"], (hd,), "f32", init), TensorSpec(n["k_norm"], (hd,), "f32", init)]
@@ -117,10 +130,12 @@ class Attention(Mixer):
         # on the device as it arrives, so that no two copies of the three are held at once
         nq, nk, nv, n = self.nq, self.nk, self.nv, self.names
         pieces = ("q", "k") if self.values_are_keys else ("q", "k", "v")
-        self.w_qkv = torch.empty((nq + nk + nv, self.D), dtype=rt.dtype, device=rt.device)
+        self.w_qkv = (torch.zeros if self.ng else torch.empty)((nq + nk + nv + self.ng, self.D), dtype=rt.dtype, device=rt.device)
+        if self.head_gate:
+            self.w_qkv[self.g_col:self.g_col + self.Hq].copy_(get(n["gate"]))
         for name, lo, hi in ((n["q"], 0, nq), (n["k"], nq, nq + nk), (n["v"], nq + nk, nq + nk + nv))[:len(pieces)]:
             self.w_qkv[lo:hi].copy_(get(name))
-        self.w_q = self.w_qkv[:nq]
+        self.w_q = self.w_qkv if self.head_gate else self.w_qkv[:nq]      # what a layer that reads another's pages multiplies with
         self.w_o = to_operand(get(n["o"]), rt)
         if self.qk_norm and self.qk_norm_weight:
             self.q_norm, self.k_norm = to_f32(get(n["q_norm"]), rt), to_f32(get(n["k_norm"]), rt)
@@ -173,7 +188,8 @@ class Attention(Mixer):
             raise ValueError("a layer that borrows another's keys cannot convolve its own")
         ops.current_tag = "attention.conv"
         tail = state["conv"] if self.taps > 1 else self._no_tail
-        return ops.short_conv(qkv, self.conv_w.shape[0], self.conv_w, self.bias, tail, ctx.req_of_token, ctx.q_start, ctx.slot_ids, ctx.R)
+        return ops.short_conv(qkv, self.conv_w.shape[0], self.conv_w, self.bias, tail, ctx.req_of_token, ctx.q_start, ctx.slot_ids, ctx.R,
+                              copy_to=self.g_col + self.ng)
 
     def _forward_flexible(self, xn, ctx, cache, state=None):
         """Any key and value widths, a window and/or chunks, mixed heads: the flexible kernels."""
@@ -185,7 +201,7 @@ class Attention(Mixer):
         M = self.maps
         q = ops.qkv_pages(qkv, self.Hq * M, self.Hkv * M, self.hd, self.vd, self.q_norm, self.k_norm, self.eps, self.pos.rotary_table(),
                           ctx.positions, ctx.req_of_token, table if write else None, cache.page_size, cache.k if write else None,
-                          cache.v if write else None, rt.dtype, v_heads=self.Hkv, bias=self.prep_bias, values_are_keys=self.values_are_keys)
+                          cache.v if write else None, rt.dtype, v_heads=self.Hkv, bias=self.prep_bias, values_are_keys=self.values_are_keys, value_norm=self.value_norm)
         ops.current_tag = "attention.keys"
         tiles = None if rt.is_fp32 or not rt.tensor_cores else ctx.query_tiles(ops.attention_flex_tile_tokens(self.Hq, self.Hkv))
         a = ops.attention_flex(None, q.view(-1, self.hd), False, cache.k, cache.v, table, ctx.req_of_token, ctx.positions, self.Hq * M,
@@ -194,6 +210,13 @@ class Attention(Mixer):
         if M > 1:                                   # a head's two maps, FP32, into the head's one result
             ops.current_tag = "attention.maps"
             a = ops.map_difference(a, self.Hq, self.vd, self.map_weight, self.eps, 1.0 - self.diff, rt.dtype)
+        return self._gated_out(a, qkv, ctx)
+
+    def _gated_out(self, a, qkv, ctx):
+        """The heads' gates (columns of the stacked product), then the output projection."""
+        if self.head_gate:
+            ops.current_tag = "attention.gate"
+            ops.gate_heads(a, self.Hq, qkv, self.g_col)
         ops.current_tag = "attention.o"
         return self._out(a, ctx)
 
@@ -222,7 +245,7 @@ class Attention(Mixer):
         # a step of a few tokens per request: the kernel that splits the keys normalises and rotates q itself and makes
         # the new keys and values (one launch less)
         in_attention = (self.prepare_in_attention and how[0] == "split" and fused_pos and self.conv_w is None and self.prep_bias is None and
-                        not self.values_are_keys and
+                        not self.values_are_keys and not self.value_norm and
                         ops.attention_mma_prepares(self.hd, self.Hq // self.Hkv, how[1][0], rotary[1] if rotary else 0, bool(rotary and rotary[2])))
         # FP32 [T, (Hq + 2 Hkv) hd] or [T, Hq hd]; for few rows possibly as split-K partials, which the next kernel sums
         ops.current_tag = "attention.qkv"
@@ -233,23 +256,22 @@ class Attention(Mixer):
             a = self._split_keys(None, cache, table, ctx, how[1],
                                  prepare={"qkv": qkv, "heads": self.Hq, "q_norm": self.q_norm, "k_norm": self.k_norm, "eps": self.eps,
                                           "rotary": rotary, "write": write})
-            ops.current_tag = "attention.o"
-            return self._out(a, ctx)
+            return self._gated_out(a, qkv, ctx)
         ops.current_tag = "attention.prepare"
         if not fused_pos:
-            qkv = self._unfused_position(qkv, ctx, write)
-            q = ops.qk_prep(qkv, self.Hq, self.Hkv, self.hd, None, None, self.eps, None, ctx.positions, ctx.req_of_token,
+            turned = self._unfused_position(qkv, ctx, write)
+            q = ops.qk_prep(turned, self.Hq, self.Hkv, self.hd, None, None, self.eps, None, ctx.positions, ctx.req_of_token,
                             table if write else None, cache.page_size, cache.k if write else None,
                             cache.v if write else None, rt.dtype)
         else:
             q = ops.qk_prep(qkv, self.Hq, self.Hkv, self.hd, self.q_norm, self.k_norm, self.eps, rotary, ctx.positions,
                             ctx.req_of_token, table if write else None, cache.page_size, cache.k if write else None,
-                            cache.v if write else None, rt.dtype, bias=self.prep_bias, values_are_keys=self.values_are_keys)
+                            cache.v if write else None, rt.dtype, bias=self.prep_bias, values_are_keys=self.values_are_keys,
+                            value_norm=self.value_norm)
         ops.current_tag = "attention.keys"
         a = self._attend(q, cache, table, ctx, how)
         # the block adds it into the stream inside its next norm (which also sums split-K partials)
-        ops.current_tag = "attention.o"
-        return self._out(a, ctx)
+        return self._gated_out(a, qkv, ctx)
 
     prepare_in_attention = True   # the kernel that splits the keys makes q and the new keys itself where it can (else qk_prep does)
     tc_min_fill = 0.5             # the tcgen05 prompt kernel runs when its CTAs (two tiles each) cover at least this share of the SMs
@@ -332,5 +354,5 @@ class Attention(Mixer):
                 k = ops.rmsnorm(k, self.k_norm, self.eps, torch.float32)
             k = k.view(T, self.Hkv, self.hd)
             self.pos.apply(k, ctx.positions)
-            parts += [k.reshape(T, nk), qkv[:, nq + nk:]]
+            parts += [k.reshape(T, nk), qkv[:, nq + nk:nq + nk + self.nv]]
         return torch.cat(parts, dim=1).contiguous()

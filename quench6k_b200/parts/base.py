@@ -20,6 +20,7 @@ under a name with the matching `register_*`; a spec.PartSpec(kind=name, params=.
                   float32 [T, D] result (or [slices, T, D] partial sums) for the block's next norm to add
   FeedForward     tensors(); bind(); forward(xn [T, D], ctx, out_f32 [T, D]) adds its result into `out`
   Block           built from (norm1, mixer, norm2, ffn); forward(h, ctx, cache, state)
+  Connection      tensors(); bind(); what ties a sublayer to a residual of several streams (base.Streams), in arrangements that have one
   EmbedAdd        tensors(); bind(); state_shape() as a mixer's; forward(h_f32 [T, D], ctx, state) adds into h in place
 """
 from __future__ import annotations
@@ -141,6 +142,49 @@ class ScaledSum:
                             bias=self.bias)
 
 
+@dataclass
+class NormedPair:
+    """A mixer's result that has not been made yet: mult * (norm(a + bias) wa + norm(b) wb), two results side by side, each over
+    its root mean square along the row.  A mixer may return it to a block that says so (StepContext.takes_pair)."""
+    a: torch.Tensor                       # FP32 [T, D], or [slices, T, D] partial sums to be added in order
+    b: torch.Tensor
+    wa: torch.Tensor
+    wb: torch.Tensor
+    mult: float
+    eps: float
+    bias: Optional[torch.Tensor] = None   # FP32 [D], added to a
+
+
+class Streams:
+    """A residual of several streams: x is FP32 [T, D] while all of them still equal the embedding output, [T, S, D] after the
+    first add.  `step` makes an add that was left (a StreamAdd or None) and reads one combination of the streams through an
+    RMS norm, in one pass over the rows."""
+
+    def __init__(self, x: torch.Tensor, count: int):
+        self.x, self.count = x, int(count)
+
+    def step(self, pending: "Optional[StreamAdd]", weights: torch.Tensor, norm, rows=None) -> torch.Tensor:
+        from .. import ops
+        self.x, out = ops.hyper_step(self.x, self.count, None if pending is None else pending.add, (weights, norm.weight, norm.eps), rows,
+                                     norm.rt.dtype)
+        return out
+
+    def total(self) -> torch.Tensor:
+        """The sum of the streams, FP32 [T, D]."""
+        return self.x * self.count if self.x.dim() == 2 else self.x.sum(1)
+
+
+@dataclass
+class StreamAdd:
+    """An add into a residual of several streams that has not been made yet: x_t <- sum_s mix[s, t] x_s + out[t] y (`add`: what
+    ops.hyper_step takes)."""
+    add: dict
+
+    def apply(self, h: Streams) -> None:
+        from .. import ops
+        h.x, _ = ops.hyper_step(h.x, h.count, self.add)
+
+
 class Tap:
     """A debugging aid: a part that is given a Tap copies small per-row results of every forward
     into it (the routed experts: each row's chosen experts and its router logits), one static
@@ -219,6 +263,10 @@ class EmbedAdd(Part):
         raise NotImplementedError
 
 
+class Connection(Part):
+    """What ties a sublayer to a residual of several streams."""
+
+
 class FeedForward(Part):
     defers_add = False                    # forward(..., defer=True) may return a WeightedRows instead of adding
 
@@ -230,15 +278,18 @@ class Block:
     takes_extra = False                   # forward(..., extra=x) adds x into the stream inside the block's first norm
 
     def __init__(self, norm1: Norm, mixer: Mixer, norm2: Optional[Norm], ffn: Optional[FeedForward],
-                 norm1b: Optional[Norm] = None, norm2b: Optional[Norm] = None, side: Optional[FeedForward] = None):
+                 norm1b: Optional[Norm] = None, norm2b: Optional[Norm] = None, side: Optional[FeedForward] = None,
+                 connect1: Optional[Connection] = None, connect2: Optional[Connection] = None):
         self.norm1, self.mixer, self.norm2, self.ffn = norm1, mixer, norm2, ffn
         self.norm1b, self.norm2b = norm1b, norm2b      # norms of the sublayers' results, in arrangements that have them
         self.side = side                               # a third sublayer fed by the model's side table, in arrangements that have one
 
+        self.connect1, self.connect2 = connect1, connect2   # ties to a residual of several streams, in arrangements that have one
+
     def parts(self):
         """(role, part) of everything that holds tensors, in the order the tensors are declared."""
         out = [("norm1", self.norm1), ("mixer", self.mixer), ("norm2", self.norm2), ("ffn", self.ffn),
-               ("norm1b", self.norm1b), ("norm2b", self.norm2b), ("side", self.side)]
+               ("norm1b", self.norm1b), ("norm2b", self.norm2b), ("side", self.side), ("connect1", self.connect1), ("connect2", self.connect2)]
         return [(k, v) for k, v in out if v is not None]
 
     def forward(self, h, ctx, cache, state, pending=None):
@@ -253,6 +304,7 @@ MIXERS: Dict[str, type] = {}
 FEED_FORWARDS: Dict[str, type] = {}
 BLOCKS: Dict[str, type] = {}
 EMBED_ADDS: Dict[str, type] = {}
+CONNECTIONS: Dict[str, type] = {}
 
 
 def _register(table: Dict[str, type], what: str):
@@ -270,6 +322,7 @@ register_mixer = _register(MIXERS, "mixer")
 register_feed_forward = _register(FEED_FORWARDS, "feed-forward")
 register_block = _register(BLOCKS, "block")
 register_embed_add = _register(EMBED_ADDS, "embedding add")
+register_connection = _register(CONNECTIONS, "connection")
 
 
 def make_part(table: Dict[str, type], what: str, spec: PartSpec, **extra):

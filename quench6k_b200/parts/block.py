@@ -3,7 +3,8 @@ the residual stream h staying FP32 (reference: crates/engine/src/flint.rs:815-10
 from __future__ import annotations
 
 from .. import ops
-from .base import Block, PostNormed, ScaledSum, WeightedRows, register_block
+from ..spec import TensorSpec
+from .base import Block, Connection, NormedPair, PostNormed, ScaledSum, StreamAdd, WeightedRows, register_block, register_connection, to_f32
 from .norm import RMSNorm
 
 
@@ -138,3 +139,70 @@ class OutNormBlock(Block):
             x = self._close(h, left, dtype)
             left = PostNormed(self.side.compute(x, ctx), self.side.norm)
         return left
+
+
+@register_connection("hyper")
+class HyperConnection(Connection):
+    """A sublayer in a residual of `streams` streams: it reads sum_s in[s] x_s, and its result y leaves every stream as
+    x_t <- sum_s mix[s, t] x_s + out[t] y.  Three stored tensors, FP32."""
+    graph_safe = True
+
+    def __init__(self, streams: int, names=None):
+        self.S = int(streams)
+        self.names = {"in": "in", "out": "out", "mix": "mix", **(names or {})}
+
+    def tensors(self):
+        n, S = self.names, self.S
+        return [TensorSpec(n["in"], (S,), "f32", ("normal", 0.5)), TensorSpec(n["out"], (S,), "f32", ("ones_plus", 0.3)),
+                TensorSpec(n["mix"], (S, S), "f32", ("normal", 0.5))]
+
+    def bind(self, get, rt):
+        if not 0 < self.S <= ops.hyper_max_streams():
+            raise ValueError(f"{self.S} streams: the kernel takes 1 to {ops.hyper_max_streams()}")
+        self.rt = rt
+        self.read, self.out, self.mix = (to_f32(get(self.names[x]), rt) for x in ("in", "out", "mix"))
+
+
+@register_block("hyper")
+class HyperBlock(Block):
+    """Sublayers in a residual of several streams (base.Streams): each reads one combination of the streams through a norm and
+    its result goes into all of them, connect1 and connect2 holding the weights.  An add, the combination the next sublayer
+    reads and its norm are one kernel; the block's last add is left to the block after it (or to the model's last norm)."""
+
+    def _read(self, h, pending, connect, norm):
+        if not isinstance(norm, RMSNorm):
+            raise TypeError("a residual of several streams is read through RMS norms")
+        return h.step(pending, connect.read, norm)
+
+    @staticmethod
+    def _add(connect, y, bias=None, weighted=None):
+        add = {"mix": connect.mix, "out": connect.out, "bias": bias}
+        if isinstance(y, NormedPair):
+            add.update(a=y.a, bias=y.bias, pair=(y.b, y.wa, y.wb, y.mult, y.eps))
+        else:
+            add["a"] = y
+        if weighted is not None:
+            add["weighted"] = (weighted.y, weighted.pair_row, weighted.weights)
+        return StreamAdd(add)
+
+    def forward(self, h, ctx, cache, state, pending=None):
+        ops.current_tag = "streams.mixer"
+        x = self._read(h, pending, self.connect1, self.norm1)
+        ctx.leave_bias = ctx.takes_pair = True            # the add takes a projection's bias and two normed results
+        ctx.left_bias = None
+        y = self.mixer.forward(x, ctx, cache, state, None)
+        ctx.leave_bias = ctx.takes_pair = False
+        if y is None:
+            raise TypeError(f"{type(self.mixer).__name__} adds into the stream itself; this arrangement needs its result")
+        if isinstance(y, NormedPair) and y.eps != self.norm1.eps:
+            from .side_by_side import made
+            y = made(y)                                   # the fused add has one eps
+        left = self._add(self.connect1, y, ctx.left_bias)
+        if self.ffn is None:
+            return left
+        ops.current_tag = "streams.ffn"
+        x = self._read(h, left, self.connect2, self.norm2)
+        if getattr(self.ffn, "defers_add", False):
+            y, rows = self.ffn.compute(x, ctx)            # (what every token shares or None, the routed rows unsummed)
+            return self._add(self.connect2, y, weighted=rows)
+        return self._add(self.connect2, self.ffn.compute(x, ctx))

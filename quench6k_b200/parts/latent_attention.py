@@ -7,7 +7,7 @@ latent space, which needs nothing but the cache: with q_h = [a_h | r_h],
 so every head attends with a query of rank + rot_dim over one shared key row per position whose first `rank` entries
 are also its value: multi-query attention over the pages, between two per-head products.
 
-Options: a sliding window (position i sees j with 0 <= i - j < window), a learned sink per head (exp(sink_h) joins the
+Options: queries through a normed low-rank vector of their own (`q_rank`: q = W_uq norm(W_dq x)), a sliding window (position i sees j with 0 <= i - j < window), a learned sink per head (exp(sink_h) joins the
 softmax denominator), either pairing of the rotation, and a layer that has no down-projection of its own but reads the
 pages another layer wrote (`borrows`: its own queries, up-projections, mask and output product).  A layer whose pages
 are read by layers with wider windows keeps them for the widest (`retain`: a window, or None for every key)."""
@@ -19,7 +19,8 @@ from . import linear
 from .base import POSITION_ENCODINGS, CacheRequest, Mixer, make_part, register_mixer, to_f32, to_operand
 
 _NAMES = {"q": "q_proj.weight", "dkv": "kv_down_proj.weight", "c_norm": "kv_norm.weight", "uk": "k_up_proj.weight",
-          "uv": "v_up_proj.weight", "out": "o_proj.weight", "sinks": "sinks"}
+          "uv": "v_up_proj.weight", "out": "o_proj.weight", "sinks": "sinks",
+          "dq": "q_down_proj.weight", "q_norm": "q_norm.weight", "uq": "q_up_proj.weight"}
 
 
 @register_mixer("latent_attention")
@@ -28,8 +29,8 @@ class LatentAttention(Mixer):
 
     def __init__(self, hidden_size: int, num_heads: int, head_dim: int, rot_dim: int, v_dim: int, kv_rank: int, scale: float, eps: float,
                  pos: PartSpec, names=None, norm_init: str = "ones", window=None, sinks: bool = False, sink_std: float = 1.0,
-                 borrows: bool = False, retain="window"):
-        """window: the sliding window's size (None: causal).  sinks: a learned number per head in the softmax denominator.
+                 borrows: bool = False, retain="window", q_rank: int = 0):
+        """q_rank: width of the queries' low-rank vector (0: queries straight from the input).  window: the sliding window's size (None: causal).  sinks: a learned number per head in the softmax denominator.
         borrows: no down-projection and no pages of its own (the model names the layer whose pages it reads).  retain:
         how long this layer's pages are kept: "window" (its own window), an integer (a wider window of a layer that
         reads them) or None (every key)."""
@@ -45,12 +46,17 @@ class LatentAttention(Mixer):
         self.retain = self.window if retain == "window" else (int(retain) if retain else None)
         if self.window is not None and self.retain is not None and self.retain < self.window:
             raise ValueError(f"pages kept for {self.retain} positions under a window of {self.window}")
+        self.q_rank = int(q_rank)
         self.names = {**_NAMES, **(names or {})}
 
     def tensors(self):
         n, H = self.names, self.H
         init = ("ones",) if self.norm_init == "ones" else ("ones_plus", 0.1)
-        out = [TensorSpec(n["q"], (H * (self.dim + self.rd), self.D))]
+        if self.q_rank:
+            out = [TensorSpec(n["dq"], (self.q_rank, self.D)), TensorSpec(n["q_norm"], (self.q_rank,), "f32", init),
+                   TensorSpec(n["uq"], (H * (self.dim + self.rd), self.q_rank))]
+        else:
+            out = [TensorSpec(n["q"], (H * (self.dim + self.rd), self.D))]
         if not self.borrows:
             out += [TensorSpec(n["dkv"], (self.rank + self.rd, self.D)), TensorSpec(n["c_norm"], (self.rank,), "f32", init)]
         out += [TensorSpec(n["uk"], (H * self.dim, self.rank)), TensorSpec(n["uv"], (H * self.vd, self.rank))]
@@ -62,10 +68,13 @@ class LatentAttention(Mixer):
         import torch
         self.rt = rt
         n, H = self.names, self.H
-        nq = H * (self.dim + self.rd)
+        nq = self.q_rank or H * (self.dim + self.rd)
         own = 0 if self.borrows else self.rank + self.rd
-        self.w_qd = torch.empty((nq + own, self.D), dtype=rt.dtype, device=rt.device)     # one product: [q | latent | shared key part]
-        self.w_qd[:nq].copy_(get(n["q"]))
+        # one product: [q (or its low-rank vector) | latent | shared key part]
+        self.w_qd = torch.empty((nq + own, self.D), dtype=rt.dtype, device=rt.device)
+        self.w_qd[:nq].copy_(get(n["dq" if self.q_rank else "q"]))
+        if self.q_rank:
+            self.q_norm, self.w_uq = to_f32(get(n["q_norm"]), rt), to_operand(get(n["uq"]), rt)
         if not self.borrows:
             self.w_qd[nq:].copy_(get(n["dkv"]))
         self.c_norm = None if self.borrows else to_f32(get(n["c_norm"]), rt)
@@ -91,10 +100,15 @@ class LatentAttention(Mixer):
         table = ctx.block_tables[cache.group]
         ops.current_tag = "latent.qkv"
         x = linear.matmul(xn, self.w_qd, rt)
+        latent = None
+        if self.q_rank:
+            ops.current_tag = "latent.queries"
+            latent = (x, self.q_rank)
+            x = linear.matmul(ops.norm_columns(x, 0, self.q_rank, self.q_norm, self.eps, rt.dtype), self.w_uq, rt)
         ops.current_tag = "latent.prepare"
         inv_freq, turn, neighbours = (None, 0, False) if self.pos.is_identity else self.pos.rotary_table()
         qn, qr = ops.latent_prep(x, H, self.dim, self.rd, self.rank, self.c_norm, self.eps, inv_freq, turn, ctx.positions,
-                                 ctx.req_of_token, table, cache.page_size, cache.k, neighbours=neighbours, write=not self.borrows)
+                                 ctx.req_of_token, table, cache.page_size, cache.k, neighbours=neighbours, write=not self.borrows, latent=latent)
         ops.current_tag = "latent.absorb"
         ql = linear.batched_matmul(qn.view(H * T, self.dim), self.w_ukT, rt, T)          # FP32 [H T, rank]
         ops.current_tag = "latent.keys"
@@ -106,4 +120,4 @@ class LatentAttention(Mixer):
         ov = linear.batched_matmul(o.view(H * T, self.rank), self.w_uv, rt, T)           # FP32 [H T, vd]
         a = ops.heads_to_rows(ov, H, rt.dtype)
         ops.current_tag = "latent.o"
-        return linear.matmul(a, self.w_o, rt, partials_ok=True)
+        return linear.matmul(a, self.w_o, rt, partials_ok=not ctx.hold_results)

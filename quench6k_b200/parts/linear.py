@@ -103,11 +103,10 @@ _uniform = {}
 
 
 def _uniform_groups(groups: int, rows_per_group: int, bm: int, device):
-    """The tile list of `groups` groups of equal size, rows group-major; made once per shape (outside any recording)."""
+    """The tile list of `groups` groups of equal size, rows group-major; made once per shape (outside any recording) and kept:
+    recorded CUDA graphs point at it."""
     key = (groups, rows_per_group, bm, str(device))
     if key not in _uniform:
-        if len(_uniform) > 512:
-            _uniform.clear()
         offsets = (torch.arange(groups + 1, dtype=torch.int32) * rows_per_group).to(device)
         _uniform[key] = ops.tile_list(offsets, groups * rows_per_group, bm)
     return _uniform[key]

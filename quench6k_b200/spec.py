@@ -29,6 +29,7 @@ class LayerSpec:
     block_params: Dict[str, Any] = field(default_factory=dict)   # constants of the arrangement (a multiplier on what it adds, ...)
     side: Optional[PartSpec] = None         # a third sublayer fed by the model's side table (arrangements that have one)
     shared_norm: bool = False               # the feed-forward reads the first norm's output: the block has no second norm
+    connection: Optional[PartSpec] = None   # what ties a sublayer to a residual of several streams (arrangements that have one)
 
 
 @dataclass
@@ -49,7 +50,7 @@ class ModelSpec:
     # what follows a layer's prefix for each of its parts (a part's own tensor names come after it)
     sub_names: Dict[str, str] = field(default_factory=lambda: {"norm1": "input_layernorm.", "mixer": "self_attn.",
                                                                 "norm2": "post_attention_layernorm.", "ffn": "mlp.",
-                                                                "side": "side."})
+                                                                "side": "side.", "connect1": "connect1.", "connect2": "connect2."})
     # executed positions before which the embedding output is added to the stream again (a span of layers run several
     # times takes its input anew at the start of every pass but the first)
     readd_embedding: Tuple[int, ...] = ()
@@ -62,14 +63,18 @@ class ModelSpec:
     # hash of the token and the one before it; its tensors' names follow embed_add_prefix
     embed_add: Optional[PartSpec] = None
     embed_add_prefix: str = "model.embed_add."
+    # a residual of several streams, all equal to the embedding output at the start and summed before the last norm (0: one
+    # plain stream); the layers' block arrangement must know of it
+    streams: int = 0
 
 
 @dataclass
 class TensorSpec:
     """A tensor a part needs.  role: 'matrix' (engine dtype: bfloat16, or float32 in the 32-bit
     path), 'f32' (always float32: norm weights, sinks), 'i32' (integer tables).
-    init: ('normal', std) | ('ones',) | ('ones_plus', std) for the random-weights mode."""
+    init: ('normal', std) | ('ones',) | ('ones_plus', std) for the random-weights mode.  A dimension of None is free: the stored
+    tensor gives it, and the part learns it when the tensor is bound (the random-weights mode cannot make such a tensor)."""
     name: str
-    shape: Tuple[int, ...]
+    shape: Tuple[Optional[int], ...]
     role: str = "matrix"
     init: Tuple = ("normal", None)         # std None -> ModelSpec.init_std

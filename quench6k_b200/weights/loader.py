@@ -36,6 +36,11 @@ class WeightError(ValueError):
         super().__init__("\n".join(lines))
 
 
+def fits(shape, declared) -> bool:
+    """Whether a stored shape is the declared one (a declared dimension of None takes any size)."""
+    return len(shape) == len(declared) and all(d is None or int(n) == int(d) for n, d in zip(shape, declared))
+
+
 def check_against(declared: List[TensorSpec], found: Dict[str, tuple]) -> None:
     """found: name -> (dtype, shape).  Raises WeightError listing every discrepancy at once."""
     want = {s.name: s for s in declared}
@@ -46,8 +51,8 @@ def check_against(declared: List[TensorSpec], found: Dict[str, tuple]) -> None:
         if n not in found:
             continue
         dt, shape = found[n]
-        if tuple(shape) != tuple(s.shape):
-            wrong.append(f"{n}: shape {list(shape)}, expected {list(s.shape)}")
+        if not fits(shape, s.shape):
+            wrong.append(f"{n}: shape {list(shape)}, expected {['any' if d is None else d for d in s.shape] if None in s.shape else list(s.shape)}")
         elif s.role == "i32" and dt not in _INTS:
             wrong.append(f"{n}: dtype {dt}, expected an integer type")
         elif s.role != "i32" and dt not in _FLOATS:
@@ -150,7 +155,7 @@ def load_folder(folder: str, declared: List[TensorSpec],
         e = index[n][1]
         shape = tuple(e.shape)
         spec = want.get(target)
-        if spec is not None and target != n and shape != tuple(spec.shape) and len(shape) >= 1 and len(spec.shape) > len(shape) \
+        if spec is not None and None not in spec.shape and target != n and shape != tuple(spec.shape) and len(shape) >= 1 and len(spec.shape) > len(shape) \
                 and shape[-1] == spec.shape[-1] and _count(shape) == _count(spec.shape):
             shape = tuple(spec.shape)                    # leading dimensions flattened in the other scheme
         found[target] = (e.dtype, shape)
@@ -191,8 +196,10 @@ def load_folder(folder: str, declared: List[TensorSpec],
         return [(index[stored_as[name]][0], stored_as[name], None)]
 
     def get(name: str) -> torch.Tensor:
-        shape = tuple(want[name].shape)
         parts = pieces(name)
+        shape = tuple(want[name].shape)
+        if None in shape:                                # a free dimension: as stored
+            shape = tuple(index[parts[0][1]][1].shape)
         dtype = index[parts[0][1]][1].dtype
         if on_device and dtype in direct:
             out = torch.empty(shape, dtype=dtype, device=device)

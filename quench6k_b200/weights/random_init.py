@@ -60,6 +60,8 @@ def standard_normal(seed: int, name: str, start: int, count: int, device) -> tor
 def make_tensor(spec: TensorSpec, seed: int, default_std: float, device="cpu", dtype: Optional[torch.dtype] = None) -> torch.Tensor:
     """One declared tensor.  Matrices are bfloat16 unless `dtype` says otherwise; 'f32' tensors are
     float32; 'i32' tensors are zeros."""
+    if None in spec.shape:
+        raise ValueError(f"tensor {spec.name}: shape {list(spec.shape)} leaves a dimension to a stored tensor; the random-weights mode needs it given")
     if spec.role == "i32":
         return torch.zeros(spec.shape, dtype=torch.int32, device=device)
     out_dtype = torch.float32 if spec.role == "f32" else (dtype or torch.bfloat16)
