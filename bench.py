@@ -285,6 +285,49 @@ def kernel_retention(args):
     return 0
 
 
+def kernel_of_gunenex(args):
+    """The kernels the Gunenex design added, alone: "delta_channel" (the delta rule with a decay per key channel, with the kernel that
+    prepares its per-token inputs; counted as gated_delta's), "time_mix" (counted as retention's, with its preparation) and
+    "hyper_step" (a block's add into four streams and the next read's norm; bytes: the streams read and written, the result read,
+    the bfloat16 row written), on one request's portion of --prefill-tokens tokens, or --batch requests of one token each."""
+    import torch
+    from quench6k_b200 import ops
+    H, G, dk, dv, D, S, dev = 16, 4, 128, 128, 2048, 4, "cuda:0"
+    decode = bool(args.batch)
+    R, n = (args.batch, 1) if decode else (1, args.prefill_tokens)
+    T = R * n
+    i32 = lambda v: torch.tensor(v, dtype=torch.int32, device=dev)
+    q_start, slots, req = i32([i * n for i in range(R + 1)]), i32(list(range(R))), i32([t // n for t in range(T)])
+    rnd = lambda *shape: torch.randn(*shape, device=dev)
+    if args.kernel == "delta_channel":
+        u, p, a = rnd(T, 2 * G * dk + H * dv), rnd(T, H), rnd(T, H * dk)
+        A_log, dt_bias, state = rnd(H) - 3.0, rnd(H * dk), torch.zeros(R, H, dv, dk, device=dev)
+        run = lambda: ops.delta_channel(u, p, 0, a, 0, A_log, dt_bias, state, req, q_start, slots, R, H, G, dk, dv, prepare=n > 16)
+        flops, nbytes = 6.0 * dk * dv * H * T, 2.0 * 4 * H * dk * dv * R + 4.0 * T * (2 * G * dk + 2 * H * dv + H * dk)
+    elif args.kernel == "time_mix":
+        r, k, v, w = (rnd(T, H * dk) * 0.1 for _ in range(4))
+        w0, bonus, state = rnd(H, dk) - 3.0, rnd(H, dk), torch.zeros(R, H, dk, dv, device=dev)
+        run = lambda: ops.time_mix(r, k, v, w, w0, bonus, state, q_start, slots, R)
+        flops, nbytes = 4.0 * dk * dv * H * T, 2.0 * 4 * H * dk * dv * R + 4.0 * T * H * (4 * dk + dv)
+    else:
+        x, y, mix, out_w, in_w, w = rnd(T, S, D), rnd(T, D), rnd(S, S) * 0.25, rnd(S), rnd(S), rnd(D)
+        run = lambda: ops.hyper_step(x, S, {"a": y, "mix": mix, "out": out_w}, (in_w, w, 1e-6), None, torch.bfloat16)
+        flops, nbytes = 2.0 * T * D * S * (S + 2), T * D * (8.0 * S + 4 + 2)
+    for _ in range(max(3, args.warmup)):
+        run()
+    torch.cuda.synchronize()
+    e0, e1 = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
+    e0.record()
+    for _ in range(args.steps):
+        run()
+    e1.record()
+    torch.cuda.synchronize()
+    ms = e0.elapsed_time(e1) / args.steps
+    print(json.dumps({"kernel": args.kernel, "requests": R, "tokens_each": n, "us": round(ms * 1e3, 1), "ns_per_token": round(ms * 1e6 / n, 1),
+                      "gflops": round(flops / ms / 1e6, 1), "gbs": round(nbytes / ms / 1e6, 1), "steps": args.steps}))
+    return 0
+
+
 def profile_ops(args, runner, cfg_d, layers, ctx, stand_at_context, rand_ids):
     """Where the time of an eager decode step (batch --batch at the context) and of a prefill step goes, launcher by
     launcher: CUDA events around every launch (quench6k_b200.ops.profile_begin/profile_end), no profiler involved.  Eager
@@ -414,7 +457,28 @@ def kitodra_config(size):
             "embedding": {"bigram": {"buckets": 65521, "mul_prev": 1000003, "mul_cur": 31}}, "layers": layers}
 
 
-DESIGNS = {"pedotar": (("pedotar", pedotar_config), ("flint_dense", flint_dense_config)),
+def gunenex_config(size):
+    """Gunenex at layer sizes that resemble a real model's: a channel delta layer with a dense feed-forward, a latent
+    attention layer, a layer of attention and time mixing side by side, and a latent layer that reads the first one's latent,
+    the last three with routed experts; eight layers (the four kinds twice), four streams."""
+    D, ff, heads, kv, rank, q_rank, E, top, eff = {"s": (1024, 4096, 8, 2, 256, 384, 32, 4, 512), "m": (2048, 8192, 16, 4, 512, 768, 64, 4, 1024)}[size]
+    moe = {"kind": "moe", "expert": {"ff": eff}, "router": {"experts": E, "top": top}}
+    delta = {"type": "channel_delta", "mlp": {"kind": "dense", "ff": ff},
+             "mixer": {"heads": heads, "kv_heads": kv, "dim": 128, "vdim": 128, "conv": 4, "decay_rank": 128, "gate_rank": 128}}
+    latent = {"type": "latent_attention", "mlp": moe,
+              "mixer": {"heads": heads, "dim": 128, "vdim": 128, "q_rank": q_rank, "kv_rank": rank, "scale": 128 ** -0.5}}
+    both = {"type": "parallel", "mlp": moe,
+            "mixer": {"left": {"heads": heads, "kv_heads": kv, "dim": 128, "vdim": 128, "scale": 128 ** -0.5, "rot": {"base": 10000.0, "dims": 128}},
+                      "right": {"heads": heads, "dim": 128, "decay_rank": 64}}}
+    layers = []
+    for rep in range(2):
+        at = len(layers)
+        layers += [delta, latent, both, dict(latent, mixer=dict(latent["mixer"], kv_from=at + 1))]
+    return {"architecture": "Gunenex", "vocab": 32768, "width": D, "streams": 4, "norm": {"eps": 1e-6}, "kv_page_size": 16, "layers": layers}
+
+
+DESIGNS = {"gunenex": (("gunenex", gunenex_config), ("sigusun", sigusun_config), ("kipedra", kipedra_config)),
+           "pedotar": (("pedotar", pedotar_config), ("flint_dense", flint_dense_config)),
            "kitodra": (("kitodra", kitodra_config), ("sigusun", sigusun_config), ("kipedra", kipedra_config)),
            "kipedra": (("kipedra", kipedra_config), ("flint_routed", flint_routed_config)),
            "sigusun": (("sigusun", sigusun_config), ("kipedra", kipedra_config), ("pedotar", pedotar_config))}
@@ -580,16 +644,17 @@ def main():
     ap.add_argument("--profile-ops", action="store_true",
                     help="instead of the benchmark line: where an eager decode step and a prefill step spend their time, launcher by "
                          "launcher (CUDA events around every launch; its own JSON line)")
-    ap.add_argument("--design", default=None, choices=["pedotar", "kipedra", "sigusun", "kitodra"],
+    ap.add_argument("--design", default=None, choices=["pedotar", "kipedra", "sigusun", "kitodra", "gunenex"],
                     help="instead of the benchmark line: prefill and decode throughput of that design beside the closest Flint model "
                          "(pedotar: dense feed-forwards; kipedra: windows and routed experts; sigusun: beside Kipedra and Pedotar; kitodra: beside Sigusun and Kipedra) at equal layer sizes (--sizes), with each "
                          "model's time launcher by launcher (its own JSON line)")
     ap.add_argument("--sizes", default="s,m", help="--design: s (width 1024) and/or m (width 2048)")
-    ap.add_argument("--kernel", default=None, choices=["attention_prefill", "gated_delta", "retention"],
+    ap.add_argument("--kernel", default=None, choices=["attention_prefill", "gated_delta", "retention", "delta_channel", "time_mix", "hyper_step"],
                     help="time one kernel alone at the configuration's head sizes instead of the model: attention_prefill runs "
                          "--prefill-tokens query tokens that end at position --context (one request, contiguous pages); gated_delta runs "
                          "the delta rule recurrence over one portion of --prefill-tokens tokens, or with --batch over that many single tokens; "
-                         "retention does the same for the retention recurrence")
+                         "retention, delta_channel and time_mix do the same for the other recurrences, hyper_step for the step between two sublayers "
+                         "of a residual of several streams")
     args = ap.parse_args()
 
     if args.impl == "reference":
@@ -614,6 +679,8 @@ def main():
         return kernel_gated_delta(args)
     if args.kernel == "retention":
         return kernel_retention(args)
+    if args.kernel in ("delta_channel", "time_mix", "hyper_step"):
+        return kernel_of_gunenex(args)
     if args.design:
         torch.cuda.set_device(0)
         return design_compare(args)

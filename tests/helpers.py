@@ -35,6 +35,35 @@ def make_model_folder(folder, name, seed=0, init_std=None):
     return cfg_d, weights
 
 
+def remembered(forward):
+    """plain(cfg, weights, tokens, forced=None): what a plain implementation's `forward` gives for one sequence, kept, so that the
+    schedules and precisions a test compares with it do not compute it again.  plain.chosen holds the experts of the last
+    call (forward.chosen, where the implementation has routed experts)."""
+    known = {}
+
+    def plain(cfg_d, weights, tokens, forced=None):
+        key = (id(weights), sum(t._version for t in weights.values()), json.dumps(cfg_d, sort_keys=True), tuple(tokens),
+               None if forced is None else tuple((p, tuple(e.reshape(-1).tolist())) for p, e in sorted(forced.items())))
+        if key not in known:
+            if len(known) > 400:
+                known.clear()
+            logits = forward(cfg_d, weights, tokens, **({"forced": forced} if forced is not None else {}))
+            known[key] = (logits, getattr(forward, "chosen", None), weights)          # the weights stay alive: their id is the key
+        logits, plain.chosen, _ = known[key]
+        return logits
+
+    return plain
+
+
+def plain_on_the_engines_experts(plain, cfg, weights, tokens, forced):
+    """(logits, choices that differ, choices): a plain implementation run on the experts the engine chose ({position: [T, k]}), and
+    how often its own choice is another."""
+    want = plain(cfg, weights, tokens)
+    differ = {p: (own.sort(-1).values != forced[p].sort(-1).values).any(-1) for p, own in plain.chosen.items()}
+    flips = sum(int(d.sum()) for d in differ.values())
+    return (plain(cfg, weights, tokens, forced) if flips else want), flips, len(tokens) * len(differ)
+
+
 def random_tokens(n, vocab, seed):
     g = torch.Generator().manual_seed(seed)
     return torch.randint(0, vocab, (n,), generator=g).tolist()

@@ -45,8 +45,7 @@ def make_folder(folder, cfg_d, seed=0, init_std=0.15, doctor=None):
         return json.load(f), weights
 
 
-def plain(cfg_d, weights, tokens, forced=None):
-    return plain_kipedra.forward(cfg_d, weights, tokens, forced=forced)
+plain = helpers.remembered(plain_kipedra.forward)
 
 
 def assert_close(got, want, dtype, what, tol=None):
@@ -78,14 +77,10 @@ def replay_and_compare(folder, cfg, weights, requests, steps, max_tokens, dtype,
     got = helpers.collect(requests, steps, outputs)
     worst, flips, positions = 0.0, 0, 0
     for rid, toks in requests.items():
-        forced = runner.routing[rid]["experts"] if routed else None
-        want = plain(cfg, weights, toks, forced)
+        want = None if routed else plain(cfg, weights, toks)
         if routed:
-            own = plain_kipedra.forward(cfg, weights, toks)
-            del own
-            for p, chosen in plain_kipedra.forward.chosen.items():
-                flips += int((chosen.sort(-1).values != forced[p].sort(-1).values).any(-1).sum())
-                positions += len(toks)
+            want, flip, n = helpers.plain_on_the_engines_experts(plain, cfg, weights, toks, runner.routing[rid]["experts"])
+            flips, positions = flips + flip, positions + n
         worst = max(worst, assert_close(got[rid], want, dtype, f"{what} {dtype} {rid}"))
     assert flips <= (0.002 if dtype == "float32" else 0.05) * positions + 1, f"{what} {dtype}: {flips} of {positions} choices of experts differ"
     print(f"{what} {dtype}: worst error {worst:.3e}, {flips} of {positions} choices of experts differ")

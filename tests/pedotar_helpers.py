@@ -4,6 +4,7 @@ import os
 
 import torch
 
+import helpers
 import plain_pedotar
 
 # Relative to the largest logit of the sequence.  float32: the engine against float64 arithmetic, every position.
@@ -39,8 +40,7 @@ def make_folder(folder, cfg_d, seed=0, init_std=0.15, doctor=None):
         return json.load(f), weights
 
 
-def plain(cfg_d, weights, tokens):
-    return plain_pedotar.forward(cfg_d, weights, tokens)
+plain = helpers.remembered(plain_pedotar.forward)
 
 
 def assert_close(got, want, dtype, what, tol=None):

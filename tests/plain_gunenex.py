@@ -46,10 +46,10 @@ def causal_conv(x, taps):
     """x [T, C], taps [C, n]: y[t] = sum_j taps[:, j] * x[t - n + 1 + j], zeros before the start."""
     T, n = x.shape[0], taps.shape[1]
     y = torch.zeros_like(x)
-    for t in range(T):
-        for j in range(n):
-            if t - n + 1 + j >= 0:
-                y[t] += taps[:, j] * x[t - n + 1 + j]
+    for j in range(n):
+        back = n - 1 - j                                                # how many tokens before the current one
+        if back < T:
+            y[back:] += taps[:, j] * x[:T - back]
     return y
 
 
@@ -64,15 +64,15 @@ def channel_delta(h, w, m, eps):
     beta = torch.sigmoid(h @ w("b").T)
     rate = softplus((h @ w("a1").T) @ w("a2").T + w("dt_bias")).view(T, H, dk)
     g = torch.exp(-torch.exp(w("A_log"))[:, None] * rate)
+    of = [head // (H // G) for head in range(H)]                     # the key head of every head
     o = torch.zeros((T, H, dv), dtype=F)
-    for head in range(H):
-        kv = head // (H // G)
-        S = torch.zeros((dk, dv), dtype=F)
-        for t in range(T):
-            S = g[t, head][:, None] * S
-            u = beta[t, head] * (v[t, head] - S.T @ k[t, kv])
-            S = S + torch.outer(k[t, kv], u)
-            o[t, head] = S.T @ q[t, kv]
+    S = torch.zeros((H, dk, dv), dtype=F)
+    for t in range(T):
+        kt, qt = k[t, of], q[t, of]
+        S = g[t][:, :, None] * S
+        u = beta[t][:, None] * (v[t] - torch.einsum("hkv,hk->hv", S, kt))
+        S = S + kt[:, :, None] * u[:, None, :]
+        o[t] = torch.einsum("hkv,hk->hv", S, qt)
     o = rms_norm(o, w("norm"), eps).reshape(T, H * dv)
     return (o * torch.sigmoid((h @ w("g1").T) @ w("g2").T)) @ w("o").T
 
@@ -86,14 +86,13 @@ def gated_attention(h, w, m, eps, sink=True):
     v = rms_norm((h @ w("v").T + w("v.b")).view(T, G, dv), None, eps)
     gate = torch.sigmoid(h @ w("g").T)
     out = torch.zeros((T, H, dv), dtype=F)
+    hidden = torch.triu(torch.ones((T, T), dtype=torch.bool), 1)      # [i, j]: position i does not see j > i
     for head in range(H):
         kv = head // (H // G)
-        for i in range(T):
-            s = (k[:i + 1, kv] @ q[i, head]) * m["scale"]
-            top = torch.maximum(s.max(), w("sink")[head]) if sink else s.max()
-            e = torch.exp(s - top)
-            den = e.sum() + (torch.exp(w("sink")[head] - top) if sink else 0.0)
-            out[i, head] = gate[i, head] * ((e / den) @ v[:i + 1, kv])
+        s = ((q[:, head] @ k[:, kv].T) * m["scale"]).masked_fill(hidden, -torch.inf)
+        if sink:                                                        # one more column, with no value
+            s = torch.cat([s, w("sink")[head].expand(T, 1)], 1)
+        out[:, head] = gate[:, head, None] * (torch.softmax(s, -1)[:, :T] @ v[:, kv])
     return out.reshape(T, H * dv) @ w("o").T + w("o.b")
 
 
@@ -107,12 +106,11 @@ def time_mixing(h, w, m, eps):
     gate = silu(mix("g") @ w("g").T)
     decay = torch.exp(-torch.exp(torch.tanh(mix("w") @ w("w1").T) @ w("w2").T + w("w0"))).view(T, H, d)
     o = torch.zeros((T, H, d), dtype=F)
-    for head in range(H):
-        S = torch.zeros((d, d), dtype=F)
-        for t in range(T):
-            kv = torch.outer(k[t, head], v[t, head])
-            o[t, head] = (S + w("u")[head][:, None] * kv).T @ r[t, head]
-            S = decay[t, head][:, None] * S + kv
+    S = torch.zeros((H, d, d), dtype=F)
+    for t in range(T):
+        kv = k[t][:, :, None] * v[t][:, None, :]
+        o[t] = torch.einsum("hkv,hk->hv", S + w("u")[:, :, None] * kv, r[t])
+        S = decay[t][:, :, None] * S + kv
     o = rms_norm(o, None, eps).reshape(T, H * d) * w("norm")
     return (o * gate) @ w("o").T
 
@@ -137,9 +135,10 @@ def latent_attention(h, w, m, eps, c):
     k = (c @ w("uk").T).view(T, H, dk)
     v = (c @ w("uv").T).view(T, H, dv)
     out = torch.zeros((T, H, dv), dtype=F)
+    hidden = torch.triu(torch.ones((T, T), dtype=torch.bool), 1)
     for head in range(H):
-        for i in range(T):
-            out[i, head] = torch.softmax((k[:i + 1, head] @ q[i, head]) * m["scale"], 0) @ v[:i + 1, head]
+        s = ((q[:, head] @ k[:, head].T) * m["scale"]).masked_fill(hidden, -torch.inf)
+        out[:, head] = torch.softmax(s, -1) @ v[:, head]
     return out.reshape(T, H * dv) @ w("o").T
 
 
