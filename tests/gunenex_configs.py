@@ -53,9 +53,9 @@ G2 = model([both((3, 3, 16, 16, 0.4, 16, 10000.0), (2, 24, 10)), delta(2, 1, 24,
             latent(2, 16, 24, 32, 40, 0.35, mlp=moe(3, 1, 16))], width=64, vocab=97, page=8, streams=2, eps=1e-6)
 
 # widths at which the bfloat16 path takes its tensor-core products and attention kernels
-G3 = model([latent(4, 64, 48, 96, 128, 0.1, mlp=ff(192)), both((4, 2, 64, 64, 0.15, 64, 50000.0), (2, 64, 16), moe(8, 2, 64)),
-            delta(4, 2, 64, 32, 4, 24, 40, moe(16, 4, 32)), latent(8, 32, 64, 64, 128, 0.15, kv_from=0, mlp=moe(4, 1, 96)),
-            both((2, 1, 128, 128, 0.1, 64, 1e6), (1, 128, 32)), delta(2, 2, 128, 64, 4, 64, 8)], width=128, vocab=384, page=16, streams=4)
+G3 = model([latent(4, 64, 48, 96, 128, 0.1, mlp=ff(192)), both((4, 2, 64, 64, 0.1, 64, 50000.0), (2, 64, 16), moe(8, 2, 64)),
+            delta(4, 2, 64, 32, 4, 24, 40, moe(10, 3, 32)), latent(8, 32, 64, 64, 128, 0.1, kv_from=0, mlp=moe(4, 1, 96)),
+            both((2, 1, 128, 128, 0.07, 64, 1e6), (1, 128, 32)), delta(2, 2, 128, 64, 4, 64, 8)], width=128, vocab=384, page=16, streams=4)
 
 # no size a multiple of 4, and nine streams: every product, norm and attention takes its general path
 G4 = model([delta(5, 5, 7, 9, 3, 3, 11, moe(7, 3, 9)), latent(3, 10, 5, 13, 17, 0.4, mlp=ff(13)), both((3, 1, 10, 7, 0.45, 6, 20.0), (5, 6, 7), moe(2, 1, 6)),

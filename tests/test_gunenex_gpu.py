@@ -251,7 +251,7 @@ ONE = {
     "latent": (2, [gc.latent(3, 8, 12, 20, 24, 0.9)]),
     "latent_one_head": (5, [gc.latent(1, 24, 6, 7, 33, 0.6)]),
     "latent_borrowed": (3, [gc.latent(2, 12, 8, 10, 20, 0.8), gc.latent(4, 6, 10, 24, 20, 0.9, kv_from=0)]),
-    "latent_tensor_cores": (3, [gc.latent(4, 32, 48, 64, 64, 0.4), gc.latent(2, 64, 32, 96, 64, 0.3, kv_from=0)]),
+    "latent_tensor_cores": (3, [gc.latent(4, 32, 48, 64, 64, 0.15), gc.latent(2, 64, 32, 96, 64, 0.1, kv_from=0)]),
     "both": (3, [gc.both((4, 2, 16, 16, 0.7, 16, 300.0), (3, 16, 6))]),
     "both_no_rotation": (2, [gc.both((2, 1, 10, 14, 0.8, 0, 10.0), (2, 24, 9))]),
     "both_many_key_heads": (6, [gc.both((3, 3, 24, 8, 0.6, 10, 5000.0), (5, 6, 4))]),
@@ -313,7 +313,7 @@ def test_a_fault_would_show(single):
         assert far(b).float().mean() > 0.1 or (a - b).abs().max() > 0.05 * a.abs().max(), "the sink left out does not show"
         assert far(changed(at={"left.g": like("left.g", 0.0)})).float().mean() > 0.15, "the heads' gates left out do not show"
         b = changed(at={"right.u": like("right.u", 0.0)})         # among the first tokens, while the state holds little
-        assert far(b[:16], slice(0, 16)).float().mean() > 0.2, "the bonus left out does not show"
+        assert far(b[:8], slice(0, 8)).float().mean() > 0.2, "the bonus left out does not show"
         assert far(changed(at={"right.mu.k": like("right.mu.k", 0.0)})).float().mean() > 0.15, "the token before does not show"
     if name.startswith("delta"):
         if cfg["layers"][0]["mixer"]["conv"] > 1:

@@ -13,6 +13,7 @@ import gunenex_helpers as gh
 import helpers
 
 pytestmark = pytest.mark.gpu
+INIT_STD = 0.1
 
 
 def draw(seed, tensor_core=False):
@@ -28,6 +29,15 @@ def draw(seed, tensor_core=False):
         experts = rng.choice([2, 3, 5, 8, 9])
         return gc.moe(experts, rng.randint(1, min(experts, 4)), rng.choice([8, 12, 24, 64]))
 
+    width = rng.choice([64, 128, 256]) if tensor_core else rng.choice([24, 40, 72, 100, 136])
+
+    def scale(dim, *inputs):
+        """A score scale at which random weights (INIT_STD) give scores of about a unit, whatever the widths."""
+        size = INIT_STD ** 2 * dim ** 0.5
+        for n in inputs:
+            size *= n ** 0.5
+        return round(rng.choice([0.4, 0.8, 1.4]) / size, 4)
+
     layers = []
     for i in range(rng.randint(1, 5)):
         kind = rng.choice(["channel_delta", "parallel", "latent_attention"])
@@ -39,17 +49,18 @@ def draw(seed, tensor_core=False):
         elif kind == "parallel":
             dim = pick([4, 6, 8, 16, 24, 40], [32, 64, 64, 128])
             vdim = dim if rng.random() < (0.7 if tensor_core else 0.4) else pick([4, 5, 8, 16, 33], [16, 48, 64])
-            layers.append(gc.both((heads, kv, dim, vdim, rng.choice([0.05, 0.2, 0.5]), rng.choice([0, 2, dim // 4 * 2, dim]), rng.choice([20.0, 10000.0, 1e6])),
+            layers.append(gc.both((heads, kv, dim, vdim, scale(dim, width, width), rng.choice([0, 2, dim // 4 * 2, dim]), rng.choice([20.0, 10000.0, 1e6])),
                                   (rng.choice([1, 2, 3, 5]), pick([4, 6, 8, 16, 24, 70], [32, 64]), rng.choice([2, 8, 11])), feed_forward()))
         else:
             lenders = [j for j, L in enumerate(layers) if L["type"] == "latent_attention" and "kv_from" not in L["mixer"]]
             j = rng.choice(lenders) if lenders and rng.random() < 0.6 else None
             rank = layers[j]["mixer"]["kv_rank"] if j is not None else pick([7, 12, 24, 50], [32, 64, 128])
-            layers.append(gc.latent(rng.choice([1, 2, 3, 5]), pick([4, 6, 8, 16, 24], [16, 32, 64]), pick([4, 5, 8, 16, 33], [16, 32, 64]), pick([5, 8, 20], [32, 64]),
-                                    rank, rng.choice([0.1, 0.3, 0.6]), kv_from=j, mlp=feed_forward()))
+            dim, q_rank = pick([4, 6, 8, 16, 24], [16, 32, 64]), pick([5, 8, 20], [32, 64])
+            layers.append(gc.latent(rng.choice([1, 2, 3, 5]), dim, pick([4, 5, 8, 16, 33], [16, 32, 64]), q_rank, rank, scale(dim, q_rank, rank), kv_from=j,
+                                    mlp=feed_forward()))
     if tensor_core:
-        return gc.model(layers, rng.choice([64, 128, 256]), rng.choice([128, 320, 1000]), rng.choice([8, 16, 32]), rng.choice([1, 2, 4]), rng.choice([1e-6, 1e-5]))
-    return gc.model(layers, rng.choice([24, 40, 72, 100, 136]), rng.choice([17, 100, 257, 1001]), rng.choice([1, 3, 4, 8, 16, 24]), rng.choice([1, 2, 3, 4, 5, 8, 10]),
+        return gc.model(layers, width, rng.choice([128, 320, 1000]), rng.choice([8, 16, 32]), rng.choice([1, 2, 4]), rng.choice([1e-6, 1e-5]))
+    return gc.model(layers, width, rng.choice([17, 100, 257, 1001]), rng.choice([1, 3, 4, 8, 16, 24]), rng.choice([1, 2, 3, 4, 5, 8, 10]),
                     rng.choice([1e-6, 1e-5, 3e-4]))
 
 
@@ -57,7 +68,7 @@ def draw(seed, tensor_core=False):
 @pytest.mark.parametrize("seed,tensor_core", [(s, False) for s in range(14)] + [(s, True) for s in range(14, 20)])
 def test_random_configuration(tmp_path, seed, tensor_core):
     cfg = draw(seed, tensor_core)
-    cfg_d, weights = gh.make_folder(str(tmp_path), cfg, seed=seed, init_std=0.1)
+    cfg_d, weights = gh.make_folder(str(tmp_path), cfg, seed=seed, init_std=INIT_STD)
     V, page = cfg["vocab"], cfg["kv_page_size"]
     rng = random.Random(100 + seed)
     reqs = {f"r{i}": helpers.random_tokens(rng.randint(3, 90), V, 7 * seed + i) for i in range(5)}
