@@ -302,7 +302,7 @@ def kernel_of_gunenex(args):
     if args.kernel == "delta_channel":
         u, p, a = rnd(T, 2 * G * dk + H * dv), rnd(T, H), rnd(T, H * dk)
         A_log, dt_bias, state = rnd(H) - 3.0, rnd(H * dk), torch.zeros(R, H, dv, dk, device=dev)
-        run = lambda: ops.delta_channel(u, p, 0, a, 0, A_log, dt_bias, state, req, q_start, slots, R, H, G, dk, dv, prepare=n > 16)
+        run = lambda: ops.delta_channel(u, p, 0, a, 0, A_log, dt_bias, state, req, q_start, slots, R, H, G, dk, dv, prepare=n > 16, single=n == 1)
         flops, nbytes = 6.0 * dk * dv * H * T, 2.0 * 4 * H * dk * dv * R + 4.0 * T * (2 * G * dk + 2 * H * dv + H * dk)
     elif args.kernel == "time_mix":
         r, k, v, w = (rnd(T, H * dk) * 0.1 for _ in range(4))

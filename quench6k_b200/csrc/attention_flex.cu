@@ -474,6 +474,19 @@ __global__ void __launch_bounds__(128) gate_heads_kernel(T* a, const float* p, i
     for (int s = 1; s < slices; ++s) z += src[s * slice_stride];
     const float g = 1.0f / (1.0f + expf(-z));
     T* mine = a + (size_t)row * n;
+    if (sizeof(T) == 2 && n % 8 == 0 && n <= 256 && (reinterpret_cast<uintptr_t>(a) & 15) == 0) {      // 16 bytes a lane
+        if (lane * 8 >= n) return;
+        uint4* at = reinterpret_cast<uint4*>(mine) + lane;
+        uint4 u = *at;
+        __nv_bfloat162* h = reinterpret_cast<__nv_bfloat162*>(&u);
+#pragma unroll
+        for (int i = 0; i < 4; ++i) {
+            const float2 f = __bfloat1622float2(h[i]);
+            h[i] = __floats2bfloat162_rn(f.x * g, f.y * g);
+        }
+        *at = u;
+        return;
+    }
     for (int d = lane; d < n; d += 32) mine[d] = from_f32<T>(to_f32(mine[d]) * g);
 }
 

@@ -5,7 +5,7 @@
 // with q and k made unit vectors per head first (q also times dk^-1/2), beta = sigmoid(b) and the decays
 // g[x] = exp(-exp(A_log) softplus(a[x] + dt_bias[x])), everything FP32.
 //
-// Tokens are taken CH = 4 at a time, counted from the start of the request's portion.  With S the state before the chunk,
+// Tokens are taken CH at a time (four; one in a step of single tokens), counted from the start of the request's portion.  With S the state before the chunk,
 // P_i = g_1 ... g_i (per channel, products within the chunk), k'_i = P_i k_i, q'_i = P_i q_i and k''_m = (g_(m+1) ... g_CH) k_m,
 //
 //     u_i = beta_i (v_i - S^T k'_i - sum_(m<i) u_m kk[m, i]),     kk[m, i] = sum_x k_m[x] k_i[x] g_(m+1)[x] ... g_i[x]
@@ -24,11 +24,10 @@
 
 namespace {
 
-constexpr int CH = 4;                 // tokens of a chunk
-constexpr int NUM = 12;               // numbers kept per token: kk [CH], kq [CH] (index: the earlier token), beta, padding
+constexpr int CHUNK = 4;              // tokens of a chunk (one in steps that bring one token per request)
+constexpr int NUM = 12;               // numbers kept per token: kk [CHUNK], kq [CHUNK] (index: the earlier token), beta, padding
 constexpr int LANES = 8, COLS = 16, THREADS = LANES * COLS;
-constexpr int TILE = 8;               // tokens staged at a time
-constexpr int STAGES = 3;
+constexpr int TILE = 16, STAGES = 2;  // prepared inputs: tokens staged at a time, tiles in flight or in use
 constexpr int MAX_DK = 256;
 
 __device__ __forceinline__ float softplus_of(float v) { return v > 20.0f ? v : log1pf(expf(v)); }
@@ -48,6 +47,7 @@ __device__ __forceinline__ void copy4(float* dst, const float* src, bool in) {
 // decay inputs, rows lda apart; b: its beta logit, rows ldb apart.  Tokens from cnt on read as zero vectors with decays of
 // one.  Results: vec + token * vec_stride + {0, 1, 2} * width (k', q', k''), cum (P), num + token * num_stride; entries from dk
 // to `padded` are zero.
+template <int CH>
 __device__ __forceinline__ void prepare_chunk(int cnt, const float* q, const float* k, size_t ldu, const float* a, size_t lda, const float* b, size_t ldb,
                                               const float* dt_bias, float rate, int dk, int padded, float* vec, size_t vec_stride, int width,
                                               float* cum, float* num, size_t num_stride) {
@@ -115,9 +115,9 @@ __device__ __forceinline__ void prepare_chunk(int cnt, const float* q, const flo
 #pragma unroll
         for (int m = 0; m < CH; ++m) {
             const float x = m < i ? warp_sum(kk[m][i]) : 0.0f, y = m <= i ? warp_sum(kq[m][i]) : 0.0f;
-            if (lane == 0) num[i * num_stride + m] = x, num[i * num_stride + CH + m] = y;
+            if (lane == 0) num[i * num_stride + m] = x, num[i * num_stride + CHUNK + m] = y;
         }
-        if (lane == 0) num[i * num_stride + 2 * CH] = beta;
+        if (lane == 0) num[i * num_stride + 2 * CHUNK] = beta;
     }
 }
 
@@ -127,6 +127,7 @@ __global__ void __launch_bounds__(128) delta_channel_prepare_kernel(const float*
                                                                     int a_col, const float* A_log, const float* dt_bias, const int* req_of_token,
                                                                     const int* q_start, float* vec, float* num, int H, int G, int dk, int dkp) {
     pdl_enter();
+    constexpr int CH = CHUNK;
     const int t = blockIdx.x, r = req_of_token[t], i = t - q_start[r], head = blockIdx.y * 4 + (threadIdx.x >> 5);
     if (i % CH || head >= H) return;
     const int cnt = min(CH, q_start[r + 1] - t), kvh = head / (H / G);
@@ -137,7 +138,7 @@ __global__ void __launch_bounds__(128) delta_channel_prepare_kernel(const float*
     // of the arithmetic that stops there
     const float rate = -expf(A_log[head]);
     if (cnt == CH) {
-        prepare_chunk(CH, ur + kvh * dk, ur + G * dk + kvh * dk, ldu, a + (size_t)t * lda + a_col + head * dk, lda, p + (size_t)t * ldp + b_col + head, ldp,
+        prepare_chunk<CH>(CH, ur + kvh * dk, ur + G * dk + kvh * dk, ldu, a + (size_t)t * lda + a_col + head * dk, lda, p + (size_t)t * ldp + b_col + head, ldp,
                       dt_bias + head * dk, rate, dk, dkp, mine, (size_t)H * 4 * dkp, dkp, mine + 3 * dkp, nums, (size_t)H * NUM);
         return;
     }
@@ -146,7 +147,7 @@ __global__ void __launch_bounds__(128) delta_channel_prepare_kernel(const float*
     float* sv = spill + (size_t)(threadIdx.x >> 5) * (CH * 3 * dkp + dkp + CH * NUM);
     float* sc = sv + CH * 3 * dkp;
     float* sn = sc + dkp;
-    prepare_chunk(cnt, ur + kvh * dk, ur + G * dk + kvh * dk, ldu, a + (size_t)t * lda + a_col + head * dk, lda, p + (size_t)t * ldp + b_col + head, ldp,
+    prepare_chunk<CH>(cnt, ur + kvh * dk, ur + G * dk + kvh * dk, ldu, a + (size_t)t * lda + a_col + head * dk, lda, p + (size_t)t * ldp + b_col + head, ldp,
                   dt_bias + head * dk, rate, dk, dkp, sv, 3 * dkp, dkp, sc, sn, NUM);
     __syncwarp();
     const int lane = threadIdx.x & 31;
@@ -159,15 +160,16 @@ __global__ void __launch_bounds__(128) delta_channel_prepare_kernel(const float*
 }
 
 // grid (H * ceil(dv / COLS), R), THREADS threads.  RPL: rows of the state per lane, a multiple of 4 (dk <= RPL LANES).
-template <int RPL, bool PREPARED>
+template <int RPL, int CH, bool PREPARED>
 __global__ void __launch_bounds__(THREADS) delta_channel_kernel(const float* u, int ldu, const float* p, int ldp, int b_col, const float* a, int lda,
                                                                 int a_col, const float* A_log, const float* dt_bias, const float* vec, const float* num,
                                                                 float* state, const int* q_start, const int* slot_ids, float* o, int H, int G, int dk,
                                                                 int dkp, int dv) {
     pdl_enter();
-    constexpr int KS = RPL * LANES, CHUNKS = TILE / CH;
+    // without prepared inputs a chunk is made and walked at a time
+    constexpr int KS = RPL * LANES, TILE = PREPARED ? ::TILE : CH, STAGES = PREPARED ? ::STAGES : 1, CHUNKS = TILE / CH;
     constexpr int STAGE = TILE * 3 * KS + CHUNKS * KS + TILE * NUM + TILE * COLS;      // floats of a stage
-    static_assert(TILE % CH == 0 && NUM >= 2 * CH + 1 && NUM % 4 == 0 && THREADS / 32 >= CHUNKS, "whole chunks, a warp per chunk");
+    static_assert(TILE % CH == 0 && NUM >= 2 * CHUNK + 1 && NUM % 4 == 0 && CH <= CHUNK, "whole chunks");
     extern __shared__ __align__(16) float sm[];
     const int col_blocks = (dv + COLS - 1) / COLS;
     const int head = blockIdx.x / col_blocks, col0 = (blockIdx.x % col_blocks) * COLS, r = blockIdx.y, kvh = head / (H / G);
@@ -194,9 +196,10 @@ __global__ void __launch_bounds__(THREADS) delta_channel_kernel(const float* u, 
         }
         S[4 * j] = s4.x, S[4 * j + 1] = s4.y, S[4 * j + 2] = s4.z, S[4 * j + 3] = s4.w;
     }
-    // rows beyond dk (and, without a preparation, tokens beyond the portion's end) read as zero
-    for (int i = threadIdx.x; i < (PREPARED ? STAGES : 1) * STAGE; i += THREADS) sm[i] = 0.0f;
-    __syncthreads();
+    if (PREPARED) {                                   // rows beyond dk read as zero
+        for (int i = threadIdx.x; i < STAGES * STAGE; i += THREADS) sm[i] = 0.0f;
+        __syncthreads();
+    }
     auto fetch = [&](int t0, int b) {                 // PREPARED: the tile at t0 on its way to buffer b
         const int nt = min(TILE, n - t0);
         if (nt > 0) {
@@ -204,16 +207,20 @@ __global__ void __launch_bounds__(THREADS) delta_channel_kernel(const float* u, 
             float* sp = sv + TILE * 3 * KS;
             float* sn = sp + CHUNKS * KS;
             float* sval = sn + TILE * NUM;
-            const int q4 = dkp / 4;
-            for (int i = threadIdx.x; i < TILE * 3 * q4; i += THREADS) {
-                const int x = i % q4, j = (i / q4) % 3, t = i / (3 * q4);
-                const bool in = t < nt;
-                copy16(sv + (t * 3 + j) * KS + 4 * x, in ? vec + (((size_t)(first + t0 + t) * H + head) * 4 + j) * dkp + 4 * x : vec, in);
-            }
-            for (int i = threadIdx.x; i < CHUNKS * q4; i += THREADS) {
-                const int x = i % q4, c = i / q4;
-                const bool in = c * CH < nt;
-                copy16(sp + c * KS + 4 * x, in ? vec + (((size_t)(first + t0 + c * CH) * H + head) * 4 + 3) * dkp + 4 * x : vec, in);
+            constexpr int K4 = KS / 4;                // a power of two
+            const int x = threadIdx.x % K4;           // the thread's place in a row of 16-byte pieces, the same in every turn
+            static_assert(THREADS % K4 == 0 || K4 % THREADS == 0, "whole rows per turn");
+            const float* src = vec + ((size_t)(first + t0) * H + head) * 4 * dkp + 4 * x;
+            if (K4 <= THREADS ? 4 * x < dkp : true) {
+#pragma unroll
+                for (int i = threadIdx.x; i < (TILE * 3 + CHUNKS) * K4; i += THREADS) {
+                    const int row = i / K4, xx = K4 <= THREADS ? x : i % K4;
+                    if (K4 > THREADS && 4 * xx >= dkp) continue;
+                    const bool cum = row >= TILE * 3;
+                    const int t = cum ? (row - TILE * 3) * CH : row / 3, j = cum ? 3 : row % 3;
+                    const bool in = t < nt;
+                    copy16((cum ? sp + (row - TILE * 3) * KS : sv + row * KS) + 4 * xx, in ? src + ((size_t)t * H * 4 + j) * dkp + 4 * (xx - x) : vec, in);
+                }
             }
             for (int i = threadIdx.x; i < TILE * NUM / 4; i += THREADS) {
                 const int t = i / (NUM / 4), x = i % (NUM / 4);
@@ -245,14 +252,13 @@ __global__ void __launch_bounds__(THREADS) delta_channel_kernel(const float* u, 
             fetch(t0 + (STAGES - 1) * TILE, b == 0 ? STAGES - 1 : b - 1);
         } else {
             __syncthreads();
-            if (warp * CH < nt) {                     // a warp per chunk
-                const int t = first + t0 + warp * CH;
+            if (warp == 0) {
+                const int t = first + t0;
                 const float* ur = u + (size_t)t * ldu;
-                prepare_chunk(min(CH, nt - warp * CH), ur + kvh * dk, ur + G * dk + kvh * dk, ldu, a + (size_t)t * lda + a_col + head * dk, lda,
-                              p + (size_t)t * ldp + b_col + head, ldp, dt_bias + head * dk, -expf(A_log[head]), dk, dk, sv + warp * CH * 3 * KS, 3 * KS, KS,
-                              sp + warp * KS, sn + warp * CH * NUM, NUM);
+                prepare_chunk<CH>(nt, ur + kvh * dk, ur + G * dk + kvh * dk, ldu, a + (size_t)t * lda + a_col + head * dk, lda,
+                              p + (size_t)t * ldp + b_col + head, ldp, dt_bias + head * dk, -expf(A_log[head]), dk, KS, sv, 3 * KS, KS, sp, sn, NUM);
             }
-            for (int i = threadIdx.x; i < nt * COLS; i += THREADS) {
+            for (int i = threadIdx.x - 32; i >= 0 && i < nt * COLS; i += THREADS - 32) {
                 const int t = i / COLS, c = col0 + i % COLS;
                 sval[i] = c < dv ? u[(size_t)(first + t0 + t) * ldu + v_at + c] : 0.0f;
             }
@@ -287,9 +293,9 @@ __global__ void __launch_bounds__(THREADS) delta_channel_kernel(const float* u, 
                 const float* nu = sn + (c0 + i) * NUM;
                 float x = sk[i], y = sq[i];
 #pragma unroll
-                for (int m = 0; m < i; ++m) x = fmaf(uu[m], nu[m], x), y = fmaf(uu[m], nu[CH + m], y);
-                uu[i] = i < cnt ? nu[2 * CH] * (sval[(c0 + i) * COLS + cl] - x) : 0.0f;
-                y = fmaf(uu[i], nu[CH + i], y);
+                for (int m = 0; m < i; ++m) x = fmaf(uu[m], nu[m], x), y = fmaf(uu[m], nu[CHUNK + m], y);
+                uu[i] = i < cnt ? nu[2 * CHUNK] * (sval[(c0 + i) * COLS + cl] - x) : 0.0f;
+                y = fmaf(uu[i], nu[CHUNK + i], y);
                 if (i < cnt && sub == 0 && col < dv) o[((size_t)(first + t0 + c0 + i) * H + head) * dv + col] = y;
             }
             const float4* p4 = reinterpret_cast<const float4*>(sp + c0 / CH * KS) + sub;
@@ -323,13 +329,14 @@ __global__ void __launch_bounds__(THREADS) delta_channel_kernel(const float* u, 
     }
 }
 
-template <int RPL, bool PREPARED>
+template <int RPL, int CH, bool PREPARED>
 void launch_delta(dim3 grid, cudaStream_t st, const float* u, int ldu, const float* p, int ldp, int b_col, const float* a, int lda, int a_col,
                   const float* A_log, const float* dt_bias, const float* vec, const float* num, float* state, const int* q_start,
                   const int* slot_ids, float* o, int H, int G, int dk, int dkp, int dv) {
     constexpr int KS = RPL * LANES;
-    const size_t smem = (size_t)(PREPARED ? STAGES : 1) * (TILE * 3 * KS + TILE / CH * KS + TILE * NUM + TILE * COLS) * sizeof(float);
-    auto kernel = delta_channel_kernel<RPL, PREPARED>;
+    constexpr int T_ = PREPARED ? TILE : CH;
+    const size_t smem = (size_t)(PREPARED ? STAGES : 1) * (T_ * 3 * KS + T_ / CH * KS + T_ * NUM + T_ * COLS) * sizeof(float);
+    auto kernel = delta_channel_kernel<RPL, CH, PREPARED>;
     if (smem > 48 * 1024) cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
     q6k_launch(kernel, grid, THREADS, smem, st, u, ldu, p, ldp, b_col, a, lda, a_col, A_log, dt_bias, vec, num, state, q_start, slot_ids, o, H, G, dk, dkp, dv);
 }
@@ -342,10 +349,11 @@ Q6K_API long long q6k_delta_channel_scratch(int H, int dk) { return (long long)H
 
 // u: FP32 [T, ldu] = [q (G heads of dk) | k | v (H heads of dv)]; p: FP32 [T, ldp] with the H beta logits from b_col; a: FP32 [T, lda]
 // with the H dk decay inputs from a_col; dt_bias: FP32 [H dk]; state: FP32 [slots, H, dv, dk]; o: FP32 [T, H dv].
-// scratch: null, or T * q6k_delta_channel_scratch(H, dk) floats on 16 bytes.
+// scratch: null, or T * q6k_delta_channel_scratch(H, dk) floats on 16 bytes.  single: no request brings more than one token (chunks
+// of one token then).
 Q6K_API int q6k_delta_channel(const float* u, int ldu, const float* p, int ldp, int b_col, const float* a, int lda, int a_col, const float* A_log,
                               const float* dt_bias, float* scratch, float* state, const int* req_of_token, const int* q_start, const int* slot_ids,
-                              float* o, int T_, int R, int H, int G, int dk, int dv, cudaStream_t st) {
+                              float* o, int T_, int R, int H, int G, int dk, int dv, int single, cudaStream_t st) {
     if (R == 0 || T_ == 0) return 0;
     Q6K_REQUIRE(R > 0 && T_ > 0 && H > 0 && G > 0 && H % G == 0 && dk > 0 && dv > 0, "delta_channel: bad sizes R=%d H=%d G=%d dk=%d dv=%d", R, H, G, dk, dv);
     Q6K_REQUIRE(dk <= MAX_DK, "delta_channel: keys of %d entries exceed the supported %d", dk, MAX_DK);
@@ -355,7 +363,7 @@ Q6K_API int q6k_delta_channel(const float* u, int ldu, const float* p, int ldp, 
     if (scratch) {
         Q6K_REQUIRE((reinterpret_cast<uintptr_t>(scratch) & 15) == 0, "delta_channel: scratch must start on 16 bytes");
         vec = scratch, num = scratch + (size_t)T_ * H * 4 * dkp;
-        const size_t smem = 4 * (size_t)(CH * 3 * dkp + dkp + CH * NUM) * sizeof(float);
+        const size_t smem = 4 * (size_t)(CHUNK * 3 * dkp + dkp + CHUNK * NUM) * sizeof(float);
         if (smem > 48 * 1024) cudaFuncSetAttribute(delta_channel_prepare_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
         q6k_launch(delta_channel_prepare_kernel, dim3(T_, (H + 3) / 4), 128, smem, st, u, ldu, p, ldp, b_col, a, lda, a_col, A_log, dt_bias, req_of_token,
                    q_start, vec, num, H, G, dk, dkp);
@@ -364,13 +372,14 @@ Q6K_API int q6k_delta_channel(const float* u, int ldu, const float* p, int ldp, 
     const dim3 grid(H * ((dv + COLS - 1) / COLS), R);
 #define DELTA_GO(R_)                                                                                                                               \
     do {                                                                                                                                           \
-        if (scratch) launch_delta<R_, true>(grid, st, u, ldu, p, ldp, b_col, a, lda, a_col, A_log, dt_bias, vec, num, state, q_start, slot_ids, o, H, G, dk, dkp, dv); \
-        else launch_delta<R_, false>(grid, st, u, ldu, p, ldp, b_col, a, lda, a_col, A_log, dt_bias, vec, num, state, q_start, slot_ids, o, H, G, dk, dkp, dv);        \
+        if (scratch) launch_delta<R_, CHUNK, true>(grid, st, u, ldu, p, ldp, b_col, a, lda, a_col, A_log, dt_bias, vec, num, state, q_start, slot_ids, o, H, G, dk, dkp, dv); \
+        else if (single) launch_delta<R_, 1, false>(grid, st, u, ldu, p, ldp, b_col, a, lda, a_col, A_log, dt_bias, vec, num, state, q_start, slot_ids, o, H, G, dk, dkp, dv); \
+        else launch_delta<R_, CHUNK, false>(grid, st, u, ldu, p, ldp, b_col, a, lda, a_col, A_log, dt_bias, vec, num, state, q_start, slot_ids, o, H, G, dk, dkp, dv);     \
     } while (0)
     if (dk <= 4 * LANES) DELTA_GO(4);
     else if (dk <= 8 * LANES) DELTA_GO(8);
     else if (dk <= 16 * LANES) DELTA_GO(16);
-    else DELTA_GO(32);
+    else DELTA_GO(MAX_DK / LANES);
 #undef DELTA_GO
     return q6k_check_launch("delta_channel");
 }

@@ -280,6 +280,62 @@ __global__ void __launch_bounds__(256) token_shift_kernel(const T* x, const floa
     }
 }
 
+// Eight values at a time as FP32 (16 bytes of bfloat16, 32 of FP32), and back.
+template <typename T> __device__ __forceinline__ void load8(const T* p, float* v);
+template <> __device__ __forceinline__ void load8<float>(const float* p, float* v) {
+    const float4 a = reinterpret_cast<const float4*>(p)[0], b = reinterpret_cast<const float4*>(p)[1];
+    v[0] = a.x, v[1] = a.y, v[2] = a.z, v[3] = a.w, v[4] = b.x, v[5] = b.y, v[6] = b.z, v[7] = b.w;
+}
+template <> __device__ __forceinline__ void load8<__nv_bfloat16>(const __nv_bfloat16* p, float* v) {
+    const uint4 u = *reinterpret_cast<const uint4*>(p);
+    const unsigned w[4] = {u.x, u.y, u.z, u.w};
+#pragma unroll
+    for (int i = 0; i < 4; ++i) v[2 * i] = __uint_as_float(w[i] << 16), v[2 * i + 1] = __uint_as_float(w[i] & 0xffff0000u);
+}
+__device__ __forceinline__ void store8(float* p, const float* v) {
+    reinterpret_cast<float4*>(p)[0] = make_float4(v[0], v[1], v[2], v[3]);
+    reinterpret_cast<float4*>(p)[1] = make_float4(v[4], v[5], v[6], v[7]);
+}
+__device__ __forceinline__ void store8(__nv_bfloat16* p, const float* v) {
+    unsigned w[4];
+#pragma unroll
+    for (int i = 0; i < 4; ++i) {
+        const __nv_bfloat162 h = __floats2bfloat162_rn(v[2 * i], v[2 * i + 1]);
+        w[i] = *reinterpret_cast<const unsigned*>(&h);
+    }
+    *reinterpret_cast<uint4*>(p) = make_uint4(w[0], w[1], w[2], w[3]);
+}
+
+// The same for rows of a multiple of eight entries that start on 16 bytes: grid (T, ceil(D / 8 / 128)), eight entries a thread.
+template <typename T>
+__global__ void __launch_bounds__(128) token_shift8_kernel(const T* x, const float* mu, int n, float* prev, const int* req_of_token, const int* q_start,
+                                                           const int* slot_ids, T* out, int T_, int D) {
+    pdl_enter();
+    const int t = blockIdx.x, i = (blockIdx.y * 128 + threadIdx.x) * 8;
+    if (i >= D) return;
+    const int r = req_of_token[t], first = q_start[r];
+    float v[8], before[8];
+    load8<T>(x + (size_t)t * D + i, v);
+    if (t == first) {
+        float* mine = prev + (size_t)slot_ids[r] * D + i;
+        float last[8];
+        load8<float>(mine, before);
+        load8<T>(x + (size_t)(q_start[r + 1] - 1) * D + i, last);
+        store8(mine, last);
+    } else {
+        load8<T>(x + (size_t)(t - 1) * D + i, before);
+    }
+#pragma unroll
+    for (int e = 0; e < 8; ++e) before[e] -= v[e];
+    for (int j = 0; j < n; ++j) {
+        float m[8], o[8];
+        load8<float>(mu + (size_t)j * D + i, m);
+#pragma unroll
+        for (int e = 0; e < 8; ++e) o[e] = fmaf(before[e], m[e], v[e]);
+        store8(out + ((size_t)j * T_ + t) * D + i, o);
+    }
+}
+
 // A warp per (token, head): w <- exp(-exp(w + w0)) in place, bonus = sum_x u[x] k[x] r[x].
 __global__ void __launch_bounds__(128) time_mix_prep_kernel(const float* r, const float* k, int ld, float* w, const float* w0, const float* u, float* bonus,
                                                             int rows, int H, int dk) {
@@ -343,6 +399,12 @@ Q6K_API int q6k_token_shift(const void* x, const float* mu, int n, float* prev, 
                             int T_, int D, int dtype, cudaStream_t st) {
     if (T_ == 0) return 0;
     Q6K_REQUIRE(T_ > 0 && D > 0 && n > 0, "token_shift: bad sizes T=%d D=%d n=%d", T_, D, n);
+    auto on16 = [](const void* p) { return (reinterpret_cast<uintptr_t>(p) & 15) == 0; };
+    if (D % 8 == 0 && on16(x) && on16(mu) && on16(prev) && on16(out)) {
+        Q6K_DISPATCH(dtype, q6k_launch(token_shift8_kernel<T>, dim3(T_, (D / 8 + 127) / 128), 128, 0, st, (const T*)x, mu, n, prev, req_of_token, q_start, slot_ids,
+                                       (T*)out, T_, D););
+        return q6k_check_launch("token_shift");
+    }
     Q6K_DISPATCH(dtype, q6k_launch(token_shift_kernel<T>, dim3(T_), 256, 0, st, (const T*)x, mu, n, prev, req_of_token, q_start, slot_ids, (T*)out, T_, D););
     return q6k_check_launch("token_shift");
 }

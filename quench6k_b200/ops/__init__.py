@@ -1630,11 +1630,12 @@ def _delta_channel_scratch(H: int, dk: int) -> int:
 
 def delta_channel(u: torch.Tensor, p: torch.Tensor, b_col: int, a: torch.Tensor, a_col: int, A_log: torch.Tensor, dt_bias: torch.Tensor,
                   state: torch.Tensor, req_of_token: torch.Tensor, q_start: torch.Tensor, slot_ids: torch.Tensor, R: int, H: int, G: int, dk: int,
-                  dv: int, prepare: bool = False) -> torch.Tensor:
+                  dv: int, prepare: bool = False, single: bool = False) -> torch.Tensor:
     """gated_delta with one decay per head and key channel: S <- diag(g) S; u = beta (v - S^T k); S <- S + k u^T; o = S^T q with
     g = exp(-exp(A_log[h]) softplus(a + dt_bias)).  a: FP32 [T, *] with the H dk decay inputs from a_col on, dt_bias: FP32
     [H dk]; the rest as in gated_delta.  prepare: a kernel of its own makes what does not depend on the state (steps with long
-    portions); else the recurrence makes it itself.  The results are the same bit for bit."""
+    portions); else the recurrence makes it itself, with the same results.  single: the caller's word that no request brings more
+    than one token."""
     _need(u, "u", torch.float32)
     _need(p, "p", torch.float32)
     _need(a, "a", torch.float32)
@@ -1648,7 +1649,8 @@ def delta_channel(u: torch.Tensor, p: torch.Tensor, b_col: int, a: torch.Tensor,
     o = torch.empty((T, H * dv), dtype=torch.float32, device=u.device)
     scratch = torch.empty(T * _delta_channel_scratch(H, dk), dtype=torch.float32, device=u.device) if prepare else None
     _call("q6k_delta_channel", _ptr(u), _i(u.stride(0)), _ptr(p), _i(p.stride(0)), _i(b_col), _ptr(a), _i(a.stride(0)), _i(a_col), _ptr(A_log), _ptr(dt_bias),
-          _ptr(scratch), _ptr(state), _ptr(req_of_token), _ptr(q_start), _ptr(slot_ids), _ptr(o), _i(T), _i(R), _i(H), _i(G), _i(dk), _i(dv), _stream())
+          _ptr(scratch), _ptr(state), _ptr(req_of_token), _ptr(q_start), _ptr(slot_ids), _ptr(o), _i(T), _i(R), _i(H), _i(G), _i(dk), _i(dv),
+          _i(1 if single else 0), _stream())
     return o
 
 

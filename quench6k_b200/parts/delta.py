@@ -123,7 +123,7 @@ class GatedDelta(Mixer):
         prepare = ctx.max_q_len > self.prepare_beyond
         if self.channel_decay:
             o = ops.delta_channel(u, p, self.b_col, low, a_col, self.A_log, self.dt_bias, state["S"], ctx.req_of_token, ctx.q_start, ctx.slot_ids,
-                                  ctx.R, self.H, self.G, self.dk, self.dv, prepare=prepare)
+                                  ctx.R, self.H, self.G, self.dk, self.dv, prepare=prepare, single=ctx.max_q_len == 1)
         else:
             o = ops.gated_delta(u, p, self.b_col, self.a_col, self.A_log, self.dt_bias, state["S"], ctx.q_start, ctx.slot_ids, ctx.R,
                                 self.H, self.G, self.dk, self.dv, prepare=prepare)

@@ -34,7 +34,7 @@ def _portions(lens, cuts, slots):
             at[i] += cuts[i][step]
 
 
-CUTS = ([[60], [17]], [[1, 2, 30, 1, 26], [15, 2]], [[40, 3, 17], [1, 1, 15]], [[4, 5, 6, 7, 20, 18], [2, 2, 2, 11]])
+CUTS = ([[60], [17]], [[1, 1, 1, 2, 29, 1, 25], [1, 1, 13, 2]], [[40, 3, 17], [1, 1, 15]], [[4, 5, 6, 7, 20, 18], [2, 2, 2, 11]])
 
 
 # ------------------------------------------------------------------------------------------------- kernels alone
@@ -73,7 +73,7 @@ def test_delta_channel_kernels_in_portions(H, G, dk, dv):
             for live, ctx, span in _portions(lens, cuts, [3, 0]):
                 cat = lambda xs: torch.cat([xs[i][span[i][0]:span[i][1]] for i in live]).contiguous().cuda()
                 o = ops.delta_channel(cat(us), cat(ps), 2, cat(decays), 1, A_log.cuda(), dt_bias.cuda(), state, ctx.req_of_token, ctx.q_start,
-                                      ctx.slot_ids, ctx.R, H, G, dk, dv, prepare=prepare)
+                                      ctx.slot_ids, ctx.R, H, G, dk, dv, prepare=prepare, single=not prepare and ctx.max_q_len == 1)
                 row = 0
                 for i in live:
                     n = span[i][1] - span[i][0]
