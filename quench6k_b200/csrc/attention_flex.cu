@@ -474,20 +474,30 @@ __global__ void __launch_bounds__(128) gate_heads_kernel(T* a, const float* p, i
     for (int s = 1; s < slices; ++s) z += src[s * slice_stride];
     const float g = 1.0f / (1.0f + expf(-z));
     T* mine = a + (size_t)row * n;
-    if (sizeof(T) == 2 && n % 8 == 0 && n <= 256 && (reinterpret_cast<uintptr_t>(a) & 15) == 0) {      // 16 bytes a lane
-        if (lane * 8 >= n) return;
-        uint4* at = reinterpret_cast<uint4*>(mine) + lane;
-        uint4 u = *at;
-        __nv_bfloat162* h = reinterpret_cast<__nv_bfloat162*>(&u);
-#pragma unroll
-        for (int i = 0; i < 4; ++i) {
-            const float2 f = __bfloat1622float2(h[i]);
-            h[i] = __floats2bfloat162_rn(f.x * g, f.y * g);
-        }
-        *at = u;
-        return;
-    }
     for (int d = lane; d < n; d += 32) mine[d] = from_f32<T>(to_f32(mine[d]) * g);
+}
+
+// The same for bfloat16 heads of a multiple of eight entries: a thread takes eight (16 bytes) and reads its head's number at
+// the same time.
+__global__ void __launch_bounds__(256) gate_heads8_kernel(__nv_bfloat16* a, const float* p, int slices, size_t slice_stride, int ld, int col, long long count,
+                                                          int H, int n8) {
+    pdl_enter();
+    const long long idx = (long long)blockIdx.x * 256 + threadIdx.x;
+    if (idx >= count) return;
+    const int row = (int)(idx / n8);
+    uint4* at = reinterpret_cast<uint4*>(a) + idx;
+    uint4 u = *at;
+    const float* src = p + (size_t)(row / H) * ld + col + row % H;
+    float z = src[0];
+    for (int s = 1; s < slices; ++s) z += src[s * slice_stride];
+    const float g = 1.0f / (1.0f + expf(-z));
+    __nv_bfloat162* h = reinterpret_cast<__nv_bfloat162*>(&u);
+#pragma unroll
+    for (int i = 0; i < 4; ++i) {
+        const float2 f = __bfloat1622float2(h[i]);
+        h[i] = __floats2bfloat162_rn(f.x * g, f.y * g);
+    }
+    *at = u;
 }
 
 // out[t] = T(x[t, col : col + n] over its root mean square times w): n columns of FP32 rows, normed on their own.  A block per row.
@@ -515,11 +525,30 @@ __global__ void __launch_bounds__(128) norm_columns_kernel(const float* x, int l
     for (int d = threadIdx.x + 128 * KEEP; d < n; d += 128) dst[d] = from_f32<T>(src[d] * inv * w[d]);
 }
 
+// The same for at most 1,024 columns that come in fours and start on 16 bytes: a thread takes four.
+template <typename T>
+__global__ void __launch_bounds__(256) norm_columns4_kernel(const float* x, int ld, int col, int n, const float* w, float eps, T* out) {
+    pdl_enter();
+    __shared__ float red[32];
+    const int d = threadIdx.x * 4;
+    const float4 v = d < n ? *reinterpret_cast<const float4*>(x + (size_t)blockIdx.x * ld + col + d) : make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+    const float4 g = d < n ? *reinterpret_cast<const float4*>(w + d) : v;
+    const float inv = rsqrtf(block_sum(fmaf(v.x, v.x, fmaf(v.y, v.y, fmaf(v.z, v.z, v.w * v.w))), red) / (float)n + eps);
+    if (d >= n) return;
+    T* dst = out + (size_t)blockIdx.x * n + d;
+    dst[0] = from_f32<T>(v.x * inv * g.x), dst[1] = from_f32<T>(v.y * inv * g.y), dst[2] = from_f32<T>(v.z * inv * g.z), dst[3] = from_f32<T>(v.w * inv * g.w);
+}
+
 }  // namespace
 
 Q6K_API int q6k_gate_heads(void* a, const float* p, int slices, long long slice_stride, int ld, int col, int T_, int H, int n, int dtype, cudaStream_t st) {
     if (T_ == 0) return 0;
     Q6K_REQUIRE(T_ > 0 && H > 0 && n > 0 && slices >= 1 && col >= 0 && col + H <= ld && (long long)T_ * H <= 0x7fffffffLL, "gate_heads: bad sizes T=%d H=%d n=%d", T_, H, n);
+    if (dtype == Q6K_BF16 && n % 8 == 0 && (reinterpret_cast<uintptr_t>(a) & 15) == 0) {
+        const long long count = (long long)T_ * H * (n / 8);
+        q6k_launch(gate_heads8_kernel, dim3((unsigned)((count + 255) / 256)), 256, 0, st, (__nv_bfloat16*)a, p, slices, (size_t)slice_stride, ld, col, count, H, n / 8);
+        return q6k_check_launch("gate_heads");
+    }
     Q6K_DISPATCH(dtype, q6k_launch(gate_heads_kernel<T>, dim3((unsigned)(((long long)T_ * H + 3) / 4)), 128, 0, st, (T*)a, p, slices, (size_t)slice_stride, ld, col,
                                    T_ * H, H, n););
     return q6k_check_launch("gate_heads");
@@ -528,6 +557,10 @@ Q6K_API int q6k_gate_heads(void* a, const float* p, int slices, long long slice_
 Q6K_API int q6k_norm_columns(const float* x, int ld, int col, int n, const float* w, float eps, void* out, int T_, int dtype, cudaStream_t st) {
     if (T_ == 0) return 0;
     Q6K_REQUIRE(T_ > 0 && n > 0 && col >= 0 && col + n <= ld && w, "norm_columns: bad sizes T=%d n=%d", T_, n);
+    if (n % 4 == 0 && n <= 1024 && ld % 4 == 0 && (reinterpret_cast<uintptr_t>(x + col) & 15) == 0 && (reinterpret_cast<uintptr_t>(w) & 15) == 0) {
+        Q6K_DISPATCH(dtype, q6k_launch(norm_columns4_kernel<T>, dim3(T_), (n / 4 + 31) / 32 * 32, 0, st, x, ld, col, n, w, eps, (T*)out););
+        return q6k_check_launch("norm_columns");
+    }
     Q6K_DISPATCH(dtype, q6k_launch(norm_columns_kernel<T>, dim3(T_), 128, 0, st, x, ld, col, n, w, eps, (T*)out););
     return q6k_check_launch("norm_columns");
 }

@@ -222,14 +222,16 @@ def test_small_kernels():
     g = torch.Generator().manual_seed(9)
     rnd = lambda *s: torch.randn(*s, generator=g)
     for dt, tol in ((torch.float32, 1e-5), (torch.bfloat16, 3e-2)):
-        a, p = rnd(5, 3 * 20).to(dt), rnd(2, 5, 11)
-        got = a.clone().cuda()
-        ops.gate_heads(got, 3, p.cuda(), 7)
-        want = a.double().view(5, 3, 20) * torch.sigmoid(p.double().sum(0)[:, 7:10])[..., None]
-        assert (got.double().cpu().view(5, 3, 20) - want).abs().max() < tol
-        for n in (13, 200, 1500):
-            x, w = rnd(4, n + 9), rnd(n)
-            assert (ops.norm_columns(x.cuda(), 5, n, w.cuda(), 1e-5, dt).double().cpu() - pg.rms_norm(x.double()[:, 5:5 + n], w.double(), 1e-5)).abs().max() < 2 * tol
+        for n in (20, 24, 136):
+            a, p = rnd(5, 3 * n).to(dt), rnd(2, 5, 11)
+            got = a.clone().cuda()
+            ops.gate_heads(got, 3, p.cuda(), 7)
+            want = a.double().view(5, 3, n) * torch.sigmoid(p.double().sum(0)[:, 7:10])[..., None]
+            assert (got.double().cpu().view(5, 3, n) - want).abs().max() < tol
+        for n, col in ((13, 5), (200, 5), (200, 8), (1500, 5), (1500, 8), (1024, 0), (4, 4)):
+            x, w = rnd(4, n + 12), rnd(n)
+            got = ops.norm_columns(x.cuda(), col, n, w.cuda(), 1e-5, dt).double().cpu()
+            assert (got - pg.rms_norm(x.double()[:, col:col + n], w.double(), 1e-5)).abs().max() < 2 * tol, (n, col)
         z = rnd(3, 6, 10)
         assert (ops.activate(z.cuda(), 7, False, "tanh", dt).double().cpu() - torch.tanh(z.double().sum(0)[:, :7])).abs().max() < tol
         o, gate, w = rnd(5, 3 * 20), rnd(5, 60), rnd(3, 20)
