@@ -22,6 +22,7 @@
 namespace {
 
 constexpr int HYPER_MAX_STREAMS = 32;
+constexpr int HYPER_PAIRS = 64;                   // routed rows of a token whose places and weights the 16-byte kernel keeps at hand
 
 struct HyperArgs {
     const float* src; int broadcast;              // [T, S, D], or [T, D] for all streams
@@ -65,10 +66,11 @@ __device__ __forceinline__ float4 summed4(const float* x, int slices, size_t str
 // S known, D a multiple of 4 and every operand on 16 bytes.  One block per row.  Shared memory: D floats for u, 2 D more
 // for the second form of y.
 template <typename T, int S>
-__global__ void __launch_bounds__(256) hyper_vec_kernel(const HyperArgs g) {
+__global__ void __launch_bounds__(256, S <= 4 ? 3 : 1) hyper_vec_kernel(const HyperArgs g) {
     pdl_enter();
     extern __shared__ __align__(16) float us[];
-    __shared__ float red[32];
+    __shared__ float red[32], pair_w[HYPER_PAIRS];
+    __shared__ int pair_at[HYPER_PAIRS];
     const int r = blockIdx.x, t = g.rows ? g.rows[r] : r, D = g.D, D4 = D >> 2;
     const size_t row4 = (size_t)t * D4;
     const bool adds = g.a || g.py || g.bias, pair = g.wb != nullptr;
@@ -79,6 +81,13 @@ __global__ void __launch_bounds__(256) hyper_vec_kernel(const HyperArgs g) {
         iw[s] = g.in_w ? g.in_w[s] : 0.0f;
 #pragma unroll
         for (int q = 0; q < S; ++q) mix[s][q] = adds ? g.mix[s * S + q] : 0.0f;
+    }
+    if (g.py) {                                                   // the token's routed rows: where they lie and their weights
+        for (int j = threadIdx.x; j < g.pairs; j += blockDim.x) {
+            pair_at[j] = g.pair_row ? g.pair_row[t * g.pairs + j] : t * g.pairs + j;
+            pair_w[j] = g.pw[t * g.pairs + j];
+        }
+        __syncthreads();
     }
     float4* ya = reinterpret_cast<float4*>(us + D);
     float4* yb = ya + D4;
@@ -117,10 +126,8 @@ __global__ void __launch_bounds__(256) hyper_vec_kernel(const HyperArgs g) {
                 if (g.bias) y = add4(y, ld4(g.bias, i));
                 if (g.py) {
                     float4 sp = f4(0.0f);
-                    for (int j = 0; j < g.pairs; ++j) {
-                        const int at = t * g.pairs + j;
-                        sp = fma4(g.pw[at], ld4(g.py, (size_t)(g.pair_row ? g.pair_row[at] : at) * D4 + i), sp);
-                    }
+#pragma unroll 4
+                    for (int j = 0; j < g.pairs; ++j) sp = fma4(pair_w[j], ld4(g.py, (size_t)pair_at[j] * D4 + i), sp);
                     y = add4(y, sp);
                 }
             }
@@ -258,7 +265,7 @@ Q6K_API int q6k_hyper_step(const float* src, int broadcast, float* dst, const fl
     Q6K_REQUIRE(smem <= 200 * 1024, "hyper_step: rows of %d do not fit shared memory", D);
     auto on16 = [](const void* p) { return (reinterpret_cast<uintptr_t>(p) & 15) == 0; };
     // which kernel runs depends on the row width, the stream count and the buffers' alignment alone, never on the step
-    const bool vec = S <= 8 && D % 4 == 0 && slice_stride % 4 == 0 && on16(src) && on16(dst) && on16(a) && on16(bias) && on16(py) && on16(b) &&
+    const bool vec = S <= 8 && pairs <= HYPER_PAIRS && D % 4 == 0 && slice_stride % 4 == 0 && on16(src) && on16(dst) && on16(a) && on16(bias) && on16(py) && on16(b) &&
                      on16(wa) && on16(wb) && on16(norm_w) && on16(out);
 #define HYPER_GO(KERNEL)                                                                                               \
     do {                                                                                                               \
