@@ -1,7 +1,7 @@
 // A residual of several streams, and what stands between two sublayers of a model that has one.  Per token the streams
 // x_1 .. x_S are FP32 rows of D; a sublayer reads one combination of them and its result goes into all of them:
 //
-//   x_t <- sum_s mix[s, t] x_s + out[t] y      all streams at once from the old ones (mix is indexed [from, to])
+//   x_t <- sum_s mix[s, t] x_s + out[t] y      (mix[s, t]: what stream s gives to stream t)
 //   u    = sum_t in[t] x_t                      with the weights of the sublayer that comes next
 //   n    = T(u * rsqrt(mean(u^2) + eps) * w)    its norm, in the operand dtype
 //

@@ -63,7 +63,7 @@ class ModelSpec:
     # hash of the token and the one before it; its tensors' names follow embed_add_prefix
     embed_add: Optional[PartSpec] = None
     embed_add_prefix: str = "model.embed_add."
-    # a residual of several streams, all equal to the embedding output at the start and summed before the last norm (0: one
+    # a residual of several streams that start as copies of the embedding output and are summed before the last norm (0: one
     # plain stream); the layers' block arrangement must know of it
     streams: int = 0
 

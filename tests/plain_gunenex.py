@@ -55,7 +55,7 @@ def causal_conv(x, taps):
 
 # ----------------------------------------------------------------------------- mixers (one sequence, positions 0..T-1)
 def channel_delta(h, w, m, eps):
-    """The gated delta rule with one decay per head and key channel, token by token."""
+    """The gated delta rule whose decay is a vector over a head's key channels, token by token."""
     T, H, G, dk, dv = h.shape[0], m["heads"], m["kv_heads"], m["dim"], m["vdim"]
     q = silu(causal_conv(h @ w("q").T, w("q.conv"))).view(T, G, dk)
     k = silu(causal_conv(h @ w("k").T, w("k.conv"))).view(T, G, dk)
@@ -167,7 +167,7 @@ def read_streams(xs, w):
 
 
 def mix_streams(xs, y, w):
-    """Every stream anew from all the old ones (mix is indexed [from, to]) and the sublayer's result."""
+    """Every stream is rebuilt from what the streams before the add give to it (mix[s, t]: stream s to stream t) and the sublayer's result."""
     n = len(xs)
     return [sum(w("mix")[s, t] * xs[s] for s in range(n)) + w("out")[t] * y for t in range(n)]
 

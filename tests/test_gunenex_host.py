@@ -208,7 +208,7 @@ def test_experts_take_their_weight_on_the_input():
 
 
 def test_one_stream_is_a_plain_residual():
-    """With one stream, in = out = mix = 1, the streams are x <- x + sublayer(norm(x)); mix is indexed [from, to]."""
+    """With one stream, in = out = mix = 1, the streams are x <- x + sublayer(norm(x)); mix[s, t] is what stream s gives to stream t."""
     one = {"in": torch.ones(1, dtype=F), "out": torch.ones(1, dtype=F), "mix": torch.ones(1, 1, dtype=F)}
     x, y = torch.randn(3, 4, dtype=F), torch.randn(3, 4, dtype=F)
     assert torch.equal(pg.read_streams([x], _w(one)), x) and torch.allclose(pg.mix_streams([x], y, _w(one))[0], x + y)
