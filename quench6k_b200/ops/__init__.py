@@ -1705,7 +1705,7 @@ def hyper_step(x: torch.Tensor, S: int, add=None, read=None, rows: Optional[torc
     """One pass over a residual of S streams.  x: FP32 [T, S, D], or [T, D] while all streams are equal.
     add = {"a", "bias", "weighted", "pair", "mix", "out"}: x_t <- sum_s mix[s, t] x_s + out[t] y for all streams at once, y = a (FP32
     [T, D] or [slices, T, D] partial sums) + bias (FP32 [D]) + weighted rows (as in `combine`), each optional; or, with pair = (b, wa, wb,
-    mult, eps), y = mult (norm(a + bias) wa + norm(b) wb).  mix: FP32 [S, S] (from, to); out: FP32 [S].
+    mult, eps), y = mult (norm(a + bias) wa + norm(b) wb).  mix: FP32 [S, S]; out: FP32 [S].
     read = (weights FP32 [S], norm weight FP32 [D], eps): the norm of sum_t weights[t] x_t in out_dtype.
     rows: read these rows only, and store no streams.  Returns (streams [T, S, D] as they then stand, or x itself when nothing was
     added or rows are picked; the norm or None)."""

@@ -1,10 +1,10 @@
 """A recurrent mixer whose inputs each mix the token with the one before it.  With x' the row before x in its request (zeros
-for the first), each of r, k, v, g, w reads x + (x' - x) mu of its own; per head, with a matrix-valued state S [dk, dk]:
+for the first), the inputs of r, k, v, g and w are five mixes x + (x' - x) mu; per head, with a matrix-valued state S [dk, dk]:
 
     o = (S + diag(u) k v^T)^T r;    S <- diag(w) S + k v^T,    w = exp(-exp(W_w2 tanh(W_w1 x_w) + w0)) per key channel
 
-so the current token enters the read-out through the bonus u and the state after it.  Each head's o is divided by its root
-mean square, the heads side by side are multiplied by a stored weight and by silu(W_g x_g), and leave through the output
+so the current token enters the read-out through the bonus u and the state after it.  A head's o is normed over its own entries
+(root mean square, no weight), the heads side by side are multiplied by a stored weight and by silu(W_g x_g), and leave through the output
 product.
 
 The four projections run as one grouped product on the engine's matrix kernels (a group per projection, rows group by
