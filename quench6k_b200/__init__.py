@@ -8,5 +8,6 @@ from .models import kipedra as _kipedra   # noqa: F401  (registers Kipedra)
 from .models import sigusun as _sigusun   # noqa: F401  (registers Sigusun)
 from .models import kitodra as _kitodra   # noqa: F401  (registers Kitodra)
 from .models import gunenex as _gunenex   # noqa: F401  (registers Gunenex)
+from .models import kodatar as _kodatar   # noqa: F401  (registers Kodatar)
 from .sampling.params import SamplingParams      # noqa: F401
 from .engine.engine import Engine, RequestOutput   # noqa: F401

@@ -7,15 +7,21 @@ namespace {
 
 // A token id -(i + 1) stands for fed[i], the i-th token the step before has sampled, which the host
 // may not have seen yet (fed: up to n_fed ids on the device).
+// The row is multiplied by `scale`; `copy` (or null) takes it `copies` times side by side in the operand dtype, rows ldc apart.
 template <typename T>
-__global__ void embed_kernel(const int* tokens, const T* table, float* h, int D, int V, const int* fed, int n_fed) {
+__global__ void embed_kernel(const int* tokens, const T* table, float* h, int D, int V, const int* fed, int n_fed, float scale, T* copy, long long ldc,
+                             int copies) {
     pdl_enter();
     const int t = blockIdx.x;
     int tok = tokens[t];
     if (tok < 0 && fed != nullptr && -tok - 1 < n_fed) tok = fed[-tok - 1];
     tok = tok < 0 ? 0 : (tok >= V ? V - 1 : tok);      // ids are validated on the host; never read outside the table
     const T* row = table + (size_t)tok * D;
-    for (int i = threadIdx.x; i < D; i += blockDim.x) h[(size_t)t * D + i] = to_f32(row[i]);
+    for (int i = threadIdx.x; i < D; i += blockDim.x) {
+        const float v = to_f32(row[i]) * scale;
+        h[(size_t)t * D + i] = v;
+        for (int c = 0; c < copies; ++c) copy[t * ldc + (size_t)c * D + i] = from_f32<T>(v);
+    }
 }
 
 // The token-pair embedding: h[t] += table[row(t)], row = (previous token * mul_prev + token * mul_cur) mod buckets (64-bit
@@ -223,10 +229,11 @@ Q6K_API int q6k_gather_rows(const void* x, const int* idx, void* out, int rows, 
 }
 
 Q6K_API int q6k_embed(const int* tokens, const void* table, float* h, int T_, int D, int V, int dtype, const int* fed, int n_fed,
-                      cudaStream_t st) {
+                      float scale, void* copy, long long ldc, int copies, cudaStream_t st) {
     if (T_ == 0) return 0;
     Q6K_REQUIRE(T_ > 0 && D > 0 && V > 0 && n_fed >= 0, "embed: bad sizes T=%d D=%d V=%d", T_, D, V);
-    Q6K_DISPATCH(dtype, q6k_launch(embed_kernel<T>, T_, 256, 0, st, tokens, (const T*)table, h, D, V, fed, n_fed););
+    Q6K_REQUIRE(copies >= 0 && (copies == 0 || (copy && ldc >= (long long)copies * D)), "embed: %d copies in rows %lld apart", copies, ldc);
+    Q6K_DISPATCH(dtype, q6k_launch(embed_kernel<T>, T_, 256, 0, st, tokens, (const T*)table, h, D, V, fed, n_fed, scale, (T*)copy, ldc, copies););
     return q6k_check_launch("embed");
 }
 

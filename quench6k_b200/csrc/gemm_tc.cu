@@ -56,6 +56,7 @@ struct Params {
     float act_limit;                   // the clamped gate's limit
     int pair_div;                      // > 0: one tile per (token, slot) pair, see q6k_gemm_tc_pairs
     int lists_old;                     // the pair list was written before the kernel launched before this one started: weights may be fetched before the wait
+    int groups;                        // pair mode: matrices there are; a pair of a higher expert number is skipped
     int n_y, n_z;                      // row tiles (or pairs; an upper bound when num_tiles is given) and K slices
     int w_once;                        // every weight tile is fetched by one CTA only (or by a few side by side): its lines may leave the L2 cache first
 };
@@ -118,6 +119,7 @@ __device__ __forceinline__ bool decode_tile(const Params& p, int t, int n_x, int
         // tile y is pair y: its expert's weights, the single input row y / pair_div, the output row y
         const int pair = p.pair_order ? p.pair_order[y] : y;
         o.g = p.tile_group[pair];
+        if ((unsigned)o.g >= (unsigned)p.groups) return false;
         o.row0 = pair / p.pair_div;
         o.row_end = o.row0 + 1;
         o.out0 = pair;
@@ -855,6 +857,7 @@ Q6K_API int q6k_gemm_tc(const void* A, long long lda, int rows_total, const void
 // are already per pair) with the weights of expert pair_expert[y] and writes output row y.
 // pair_order (int32 [pairs] or null): the order in which the pairs are worked on; sorted by expert
 // it lets the tiles of one expert run side by side and find its weights in L2.
+// A pair whose expert number is not below `groups` (an expert without matrices) is skipped.
 // epilogue: 0 store FP32, 2 SwiGLU -> bfloat16.
 // K slices of a pair product: only when the pairs are so few that most SMs would have no tile.
 static int pair_splits(int pairs, int N, int K) {
@@ -910,6 +913,7 @@ Q6K_API int q6k_gemm_tc_pairs(const void* A, long long lda, int a_rows, const vo
     p.kb_per_split = (kb + splits - 1) / splits;
     p.partial = partial, p.tickets = tickets;
     p.pair_div = pair_div;
+    p.groups = groups;
     p.pair_order = pair_order;
     p.lists_old = lists_old;
     p.w_once = 1;                          // a pair's weight tile is shared with the few pairs of the same expert, which run side by side

@@ -465,7 +465,7 @@ __global__ void finish_rank_kernel(const int* sel_e, const int* chunk_base, cons
 // The same with the copy of the pair's input row: out[row, :] = x[pair / k, :] (rows of vec_per_row 16-byte words), a
 // block per pair.
 __global__ void finish_rank_gather_kernel(const int* sel_e, const int* chunk_base, const int* offsets,
-                                          int k, int E, int* pair_row, int* row_token, const uint4* x,
+                                          int k, int E, int live, int* pair_row, int* row_token, const uint4* x,
                                           uint4* out, int vec_per_row) {
     pdl_enter();
     const int p = blockIdx.x;
@@ -473,6 +473,7 @@ __global__ void finish_rank_gather_kernel(const int* sel_e, const int* chunk_bas
     const int row = offsets[e] + chunk_base[(p / PERM_CHUNK) * E + e] + pair_row[p];
     __syncthreads();                                     // every thread has read the rank before thread 0 replaces it
     if (threadIdx.x == 0) pair_row[p] = row, row_token[row] = p / k;
+    if (e >= live) return;                               // an expert without matrices reads no row
     const size_t src = (size_t)(p / k) * vec_per_row, dst = (size_t)row * vec_per_row;
     for (int i = threadIdx.x; i < vec_per_row; i += blockDim.x) out[dst + i] = x[src + i];
 }
@@ -481,7 +482,7 @@ __global__ void finish_rank_gather_kernel(const int* sel_e, const int* chunk_bas
 // scan over the experts of their totals (E + 1 entries).  One block.
 __device__ void tiles_in_block(const int* offsets, int G, int bm, int* tile_group, int* tile_row0, int* num_tiles, int max_tiles);
 
-__global__ void offsets_kernel(int* counts, int chunks, int E, int* offsets, int bm, int* tile_group, int* tile_row0, int* num_tiles,
+__global__ void offsets_kernel(int* counts, int chunks, int E, int live, int* offsets, int bm, int* tile_group, int* tile_row0, int* num_tiles,
                                int max_tiles) {
     pdl_enter();
     __shared__ int part[1024];
@@ -528,7 +529,7 @@ __global__ void offsets_kernel(int* counts, int chunks, int E, int* offsets, int
     }
     if (tile_group != nullptr) {
         __syncthreads();                       // this block's offsets are complete and visible to it
-        tiles_in_block(offsets, E, bm, tile_group, tile_row0, num_tiles, max_tiles);
+        tiles_in_block(offsets, live, bm, tile_group, tile_row0, num_tiles, max_tiles);
     }
 }
 
@@ -675,7 +676,7 @@ Q6K_API int q6k_moe_permute(const int* sel_e, int pairs, int k, int E, int* scra
     Q6K_REQUIRE(chunks <= 65535, "moe_permute: %d pairs exceed the grid limit", pairs);
     const dim3 grid((E + 7) / 8, chunks);
     q6k_launch(count_kernel, grid, 256, 0, st, sel_e, pairs, E, scratch);
-    q6k_launch(offsets_kernel, 1, 256, 0, st, scratch, chunks, E, offsets, 0, (int*)nullptr, (int*)nullptr, (int*)nullptr, 0);
+    q6k_launch(offsets_kernel, 1, 256, 0, st, scratch, chunks, E, E, offsets, 0, (int*)nullptr, (int*)nullptr, (int*)nullptr, 0);
     q6k_launch(rank_kernel, grid, 256, 0, st, sel_e, scratch, offsets, pairs, k, E, pair_row, row_token);
     return q6k_check_launch("moe_permute");
 }
@@ -683,11 +684,13 @@ Q6K_API int q6k_moe_permute(const int* sel_e, int pairs, int k, int E, int* scra
 // The permutation and the list of row tiles of bm rows (tile_group, tile_row0: max_tiles entries; num_tiles: 1) in
 // three launches (the block that makes the offsets also makes the tile list).
 // x != null: the pairs' input rows (row_bytes bytes each, a multiple of 16; x: [pairs / k rows]) are copied into
-// gathered[row] by the launch that finishes the ranks.
-Q6K_API int q6k_moe_plan(const int* sel_e, int pairs, int k, int E, int* scratch, int* offsets, int* pair_row, int* row_token, int bm,
+// gathered[row] by the launch that finishes the ranks.  Experts from `live` on have no matrices: their pairs come last and get
+// neither tiles nor copies.
+Q6K_API int q6k_moe_plan(const int* sel_e, int pairs, int k, int E, int live, int* scratch, int* offsets, int* pair_row, int* row_token, int bm,
                          int* tile_group, int* tile_row0, int* num_tiles, int max_tiles, const void* x, void* gathered, int row_bytes,
                          cudaStream_t st) {
     if (pairs == 0) return 0;
+    Q6K_REQUIRE(live > 0 && live <= E, "moe_plan: %d of %d experts have matrices", live, E);
     Q6K_REQUIRE(pairs > 0 && k > 0 && E > 0 && bm > 0 && max_tiles > 0, "moe_plan: bad sizes pairs=%d k=%d E=%d bm=%d", pairs, k, E, bm);
     const int chunks = (pairs + PERM_CHUNK - 1) / PERM_CHUNK;
     Q6K_REQUIRE(chunks <= 65535, "moe_plan: %d pairs exceed the grid limit", pairs);
@@ -695,9 +698,9 @@ Q6K_API int q6k_moe_plan(const int* sel_e, int pairs, int k, int E, int* scratch
                 "moe_plan: rows of %d bytes cannot be gathered (multiples of 16 bytes, 16-byte aligned buffers)", row_bytes);
     if (E <= COUNT_RANK_MAX_E) {
         q6k_launch(count_rank_kernel, chunks, PERM_CHUNK, (size_t)32 * E, st, sel_e, pairs, E, scratch, pair_row);
-        q6k_launch(offsets_kernel, 1, 256, 0, st, scratch, chunks, E, offsets, bm, tile_group, tile_row0, num_tiles, max_tiles);
+        q6k_launch(offsets_kernel, 1, 256, 0, st, scratch, chunks, E, live, offsets, bm, tile_group, tile_row0, num_tiles, max_tiles);
         if (x)
-            q6k_launch(finish_rank_gather_kernel, pairs, 128, 0, st, sel_e, scratch, offsets, k, E, pair_row, row_token, (const uint4*)x,
+            q6k_launch(finish_rank_gather_kernel, pairs, 128, 0, st, sel_e, scratch, offsets, k, E, live, pair_row, row_token, (const uint4*)x,
                        (uint4*)gathered, row_bytes / 16);
         else
             q6k_launch(finish_rank_kernel, (pairs + 255) / 256, 256, 0, st, sel_e, scratch, offsets, pairs, k, E, pair_row, row_token);
@@ -705,7 +708,7 @@ Q6K_API int q6k_moe_plan(const int* sel_e, int pairs, int k, int E, int* scratch
     }
     const dim3 grid((E + 7) / 8, chunks);
     q6k_launch(count_kernel, grid, 256, 0, st, sel_e, pairs, E, scratch);
-    q6k_launch(offsets_kernel, 1, 256, 0, st, scratch, chunks, E, offsets, bm, tile_group, tile_row0, num_tiles, max_tiles);
+    q6k_launch(offsets_kernel, 1, 256, 0, st, scratch, chunks, E, live, offsets, bm, tile_group, tile_row0, num_tiles, max_tiles);
     q6k_launch(rank_kernel, grid, 256, 0, st, sel_e, scratch, offsets, pairs, k, E, pair_row, row_token);
     if (x) {
         q6k_launch(gather_pairs_kernel, pairs, 128, 0, st, (const uint4*)x, row_token, (uint4*)gathered, row_bytes / 16);

@@ -150,13 +150,18 @@ __global__ void activate_kernel(const float* x, int slices, size_t slice_stride,
     out[idx] = from_f32<T>(gated ? z * at(r * ldx + I + i) : z);
 }
 
-// One warp per token: scores s = sigmoid(logits), the k largest of s + bias (ties to the lower index), weights
-// s / (sum of the chosen s + 1e-20) * scale, or s * scale when renorm is 0; squared at the end when `power` is 2.  logits: [slices, T, E], summed in order.
+// One warp per token: scores s = sigmoid(logits), or the softmax over all E of them; the k largest of s + bias (ties to the
+// lower index), weights s / (sum of the chosen s + 1e-20) * scale, or s * scale when renorm is 0; squared at the end when `power`
+// is 2.  logits: [slices, T, ld], summed in order; the first E columns are the experts'.
 // groups > 1: the experts form `groups` equal groups of neighbours; a group's worth is the sum of its two largest choice
-// values (its one value, if it has one expert), and only experts of the `keep` groups of most worth (ties to the lower
-// index) can be chosen.  Shared memory: E floats a warp (the choice values), E more (the scores) and `groups` more.
-__global__ void route_biased_kernel(const float* logits, int slices, size_t slice_stride, const float* bias, float scale, int T_, int E, int k,
-                                    int* sel_e, float* sel_w, int renorm, int groups, int keep, int power) {
+// values (its one value, if it has one expert), or with `best_worth` its largest one, and only experts of the `keep` groups of
+// most worth (ties to the lower index) can be chosen.
+// id_w (or null): the last `identity` experts answer their input; their weights leave as zero and their sum is id_w[t].
+// gate (or null): gate[t] = sigmoid of column E.
+// Shared memory: E floats a warp (the choice values), E more (the scores) and `groups` more.
+__global__ void route_biased_kernel(const float* logits, int slices, size_t slice_stride, int ld, const float* bias, float scale, int T_, int E, int k,
+                                    int* sel_e, float* sel_w, int renorm, int groups, int keep, int power, int softmax, int best_worth, int identity,
+                                    float* id_w, float* gate) {
     pdl_enter();
     extern __shared__ float sc[];
     const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, warps = blockDim.x >> 5;
@@ -165,12 +170,35 @@ __global__ void route_biased_kernel(const float* logits, int slices, size_t slic
     float* choice = sc + (size_t)warp * (2 * E + groups);
     float* score = choice + E;
     float* worth = score + E;
-    for (int e = lane; e < E; e += 32) {
-        float z = logits[(size_t)t * E + e];
-        for (int s = 1; s < slices; ++s) z += logits[s * slice_stride + (size_t)t * E + e];
-        const float sg = 1.0f / (1.0f + expf(-z));
-        score[e] = sg;
-        choice[e] = bias ? sg + bias[e] : sg;
+    auto logit = [&](int e) {
+        float z = logits[(size_t)t * ld + e];
+        for (int s = 1; s < slices; ++s) z += logits[s * slice_stride + (size_t)t * ld + e];
+        return z;
+    };
+    if (gate && lane == 0) gate[t] = 1.0f / (1.0f + expf(-logit(E)));
+    if (softmax) {
+        float top = -INFINITY, total = 0.0f;
+        for (int e = lane; e < E; e += 32) {
+            score[e] = logit(e);
+            top = fmaxf(top, score[e]);
+        }
+        top = warp_max(top);
+        for (int e = lane; e < E; e += 32) {
+            score[e] = expf(score[e] - top);
+            total += score[e];
+        }
+        total = warp_sum(total);
+        for (int e = lane; e < E; e += 32) {
+            const float s = score[e] / total;
+            score[e] = s;
+            choice[e] = bias ? s + bias[e] : s;
+        }
+    } else {
+        for (int e = lane; e < E; e += 32) {
+            const float sg = 1.0f / (1.0f + expf(-logit(e)));
+            score[e] = sg;
+            choice[e] = bias ? sg + bias[e] : sg;
+        }
     }
     __syncwarp();
     if (groups > 1 && keep < groups) {
@@ -182,7 +210,7 @@ __global__ void route_biased_kernel(const float* logits, int slices, size_t slic
                 if (c > a) b = a, a = c;
                 else if (c > b) b = c;
             }
-            worth[g] = per > 1 ? a + b : a;
+            worth[g] = per > 1 && !best_worth ? a + b : a;
         }
         __syncwarp();
         for (int j = 0; j < keep; ++j) {                                       // the kept groups are marked by +inf
@@ -237,9 +265,17 @@ __global__ void route_biased_kernel(const float* logits, int slices, size_t slic
     const int last = lane < k ? ((k - 1 - lane) >> 5) * 32 + lane : -1;
     if (last >= 0) sel_w[(size_t)t * k + last] = mine, sel_e[(size_t)t * k + last] = mine_e;
     __syncwarp();
+    float kept = 0.0f;
     for (int j = lane; j < k; j += 32) {
         const float v = sel_w[(size_t)t * k + j] / den * scale;
-        sel_w[(size_t)t * k + j] = power == 2 ? v * v : v;
+        const float v2 = power == 2 ? v * v : v;
+        const bool same = id_w && sel_e[(size_t)t * k + j] >= E - identity;          // this lane wrote the entry itself
+        sel_w[(size_t)t * k + j] = same ? 0.0f : v2;
+        kept += same ? v2 : 0.0f;
+    }
+    if (id_w) {
+        kept = warp_sum(kept);
+        if (lane == 0) id_w[t] = kept;
     }
 }
 
@@ -274,16 +310,19 @@ Q6K_API int q6k_activate(const float* x, int slices, long long slice_stride, int
     return q6k_check_launch("activate");
 }
 
-Q6K_API int q6k_route_biased(const float* logits, int slices, const float* bias, float scale, int T_, int E, int k, int* sel_e, float* sel_w,
-                             int renorm, int groups, int keep, int power, cudaStream_t st) {
+Q6K_API int q6k_route_biased(const float* logits, int slices, int ld, const float* bias, float scale, int T_, int E, int k, int* sel_e, float* sel_w,
+                             int renorm, int groups, int keep, int power, int softmax, int best_worth, int identity, float* id_w, float* gate,
+                             cudaStream_t st) {
     if (T_ == 0) return 0;
-    Q6K_REQUIRE(T_ > 0 && E > 0 && k > 0 && k <= E && slices >= 1, "route_biased: bad sizes T=%d E=%d k=%d slices=%d", T_, E, k, slices);
+    Q6K_REQUIRE(T_ > 0 && E > 0 && k > 0 && k <= E && slices >= 1 && ld >= E + (gate ? 1 : 0), "route_biased: bad sizes T=%d E=%d k=%d slices=%d ld=%d", T_, E, k,
+                slices, ld);
     Q6K_REQUIRE(E <= 4096, "route_biased: %d experts exceed the supported 4096", E);
     Q6K_REQUIRE(groups >= 1 && E % groups == 0 && keep >= 1 && keep <= groups && k <= keep * (E / groups),
                 "route_biased: %d experts in %d groups, %d kept, %d chosen", E, groups, keep, k);
     Q6K_REQUIRE(power == 1 || power == 2, "route_biased: weights to the power %d", power);
+    Q6K_REQUIRE(identity >= 0 && identity <= E && (identity == 0 || id_w), "route_biased: %d of %d experts answer their input", identity, E);
     const int warps = E <= 1024 ? 4 : 1;
     q6k_launch(route_biased_kernel, (T_ + warps - 1) / warps, warps * 32, (size_t)warps * (2 * E + groups) * sizeof(float), st, logits, slices,
-               (size_t)T_ * E, bias, scale, T_, E, k, sel_e, sel_w, renorm, groups, keep, power);
+               (size_t)T_ * ld, ld, bias, scale, T_, E, k, sel_e, sel_w, renorm, groups, keep, power, softmax, best_worth, identity, id_w, gate);
     return q6k_check_launch("route_biased");
 }

@@ -52,6 +52,8 @@ class StepContext:
     left_bias: Optional[torch.Tensor] = None
     takes_pair: bool = False                      # a block whose add can norm two results side by side sets it: a mixer may then return a
                                                   # parts.base.NormedPair instead of making the sum itself
+    takes_mixture: bool = False                   # a block whose norm sums everything a routed feed-forward leaves sets it: the
+                                                  # feed-forward may then return a parts.base.Mixture instead of making the sum
     position: int = 0                             # the executed position (index into the model's order) whose block is running
     side_rows: Optional[torch.Tensor] = None      # FP32 [T, columns]: the tokens' rows of the model's side table, if it has one
 

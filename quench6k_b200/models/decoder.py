@@ -13,7 +13,8 @@ import torch
 
 from .. import ops
 from ..parts import linear
-from ..parts.base import (BLOCKS, CONNECTIONS, EMBED_ADDS, FEED_FORWARDS, MIXERS, NORMS, CacheRequest, LayerCache, Runtime, Streams, WeightedRows, make_part,
+from ..parts.base import (BLOCKS, CONNECTIONS, EMBED_ADDS, FEED_FORWARDS, MIXERS, NORMS, PASS_ENTRIES, CacheRequest, LayerCache, PostNormed, Runtime, Streams,
+                          WeightedRows, make_part,
                           to_operand)
 from ..spec import ModelSpec, TensorSpec
 
@@ -56,6 +57,10 @@ class DecoderModel:
             raise ValueError("readd_embedding names a position outside 1..executed layers - 1")
         if spec.streams and self.readd:
             raise ValueError("the embedding output is not added again to a residual of several streams")
+        self.pass_entry = make_part(PASS_ENTRIES, "entry of a pass", spec.pass_entry, hidden_size=D) if spec.pass_entry is not None else None
+        self.pass_number = {p: n for n, p in enumerate(spec.pass_starts)} if self.pass_entry is not None else {}
+        if any(not 0 <= p < len(self.order) for p in self.pass_number) or (spec.streams and self.pass_number):
+            raise ValueError("pass_starts names a position outside the executed layers, or the residual has several streams")
         self.rt: Optional[Runtime] = None
 
     # ------------------------------------------------------------------ declaration
@@ -68,6 +73,8 @@ class DecoderModel:
             out += [TensorSpec(s.embed_norm_prefix + t.name, t.shape, t.role, t.init) for t in self.embed_norm.tensors()]
         if s.side_table is not None:
             out.append(TensorSpec(s.side_table[0], (s.vocab_size, s.side_table[1])))
+        if self.pass_entry is not None:
+            out += [TensorSpec(s.pass_entry_prefix + t.name, t.shape, t.role, t.init) for t in self.pass_entry.tensors()]
         for ls, b in zip(s.layers, self.blocks):
             for sub, part in b.parts():
                 out += [TensorSpec(ls.prefix + s.sub_names[sub] + t.name, t.shape, t.role, t.init) for t in part.tensors()]
@@ -90,7 +97,7 @@ class DecoderModel:
         return [self.blocks[i].mixer.state_shape() for i in self.order] + ([self.embed_add.state_shape()] if self.embed_add is not None else [])
 
     def graph_safe(self) -> bool:
-        parts = [self.final_norm] + [x for x in (self.embed_norm, self.embed_add) if x is not None]
+        parts = [self.final_norm] + [x for x in (self.embed_norm, self.embed_add, self.pass_entry) if x is not None]
         for b in self.blocks:
             parts += [part for _, part in b.parts()]
         return all(getattr(x, "graph_safe", False) for x in parts)
@@ -105,6 +112,8 @@ class DecoderModel:
         if self.embed_norm is not None:
             self.embed_norm.bind(lambda n: get(s.embed_norm_prefix + n), rt)
         self.side_table = to_operand(get(s.side_table[0]), rt) if s.side_table is not None else None
+        if self.pass_entry is not None:
+            self.pass_entry.bind(lambda n: get(s.pass_entry_prefix + n), rt)
         for ls, b in zip(s.layers, self.blocks):
             for sub, part in b.parts():
                 pre = ls.prefix + s.sub_names[sub]
@@ -118,13 +127,23 @@ class DecoderModel:
         """Runs the tokens of `ctx` through the executed layers; returns FP32 logits
         [len(ctx.logit_rows), vocab] or None when no row is wanted."""
         ops.current_tag = "embedding"
-        h = ops.embed(ctx.token_ids, self.embed, fed=ctx.fed)
+        # the products that open a pass read the stream beside the embedding output: both side by side in one buffer, which
+        # the embedding kernel fills itself unless something more is added to the embedding output
+        operand, D = None, self.spec.hidden_size
+        direct = self.embed_add is None and self.embed_norm is None
+        if self.pass_number:
+            operand = torch.empty((ctx.T, self.pass_entry.operand_width()), dtype=self.rt.dtype, device=self.rt.device)
+        h = ops.embed(ctx.token_ids, self.embed, fed=ctx.fed, scale=self.spec.embed_scale,
+                      copy=None if operand is None or not direct else operand if 0 in self.pass_number else operand[:, -D:])
         if self.embed_add is not None:
             ops.current_tag = "embedding.add"
             self.embed_add.forward(h, ctx, states[len(self.order)])
         if self.embed_norm is not None:
             ops.current_tag = "norm.embedding"
             self.embed_norm.normalize(h)
+        if operand is not None and not direct:
+            for part in (operand[:, :D], operand[:, -D:]):
+                ops.layernorm(h, None, None, 0.0, self.rt.dtype, raw=part)
         if self.side_table is not None:
             ops.current_tag = "embedding.side"
             ctx.side_rows = ops.embed(ctx.token_ids, self.side_table, fed=ctx.fed)
@@ -135,6 +154,12 @@ class DecoderModel:
         for p, i in enumerate(self.order):
             ctx.position = p
             block = self.blocks[i]
+            if p in self.pass_number:
+                ops.current_tag = "pass.stream"
+                if p > 0:
+                    self._write_stream(h, pending, operand[:, :D])
+                ops.current_tag = "pass.product"
+                pending = self.pass_entry.open(h, operand, self.pass_number[p])
             if p in self.readd:
                 if block.takes_extra:
                     pending = block.forward(h, ctx, caches[p], states[p], pending, extra=h0)
@@ -151,12 +176,23 @@ class DecoderModel:
             xn = h.step(pending, self.stream_sum, self.final_norm, rows=ctx.logit_rows)
             ops.current_tag = "lm_head"
             return linear.matmul(xn, self.head, self.rt)
-        # an add that is left: the last norm makes it if it can (it normalises picked rows only, so a sublayer result that
-        # passes a norm of its own is added first, for all rows)
-        if pending is not None and not (isinstance(pending, WeightedRows) and self.final_norm.fuses_weighted_rows):
+        # an add that is left: the last norm makes it if it can (for the rows it normalises)
+        if pending is not None and not (isinstance(pending, WeightedRows) and self.final_norm.fuses_weighted_rows
+                                        or isinstance(pending, PostNormed) and self.final_norm.fuses_picked_rows and type(pending.norm) is type(self.final_norm)
+                                        and pending.norm.eps == self.final_norm.eps):
             pending.apply(h)
             pending = None
         ops.current_tag = "norm.final"
         xn = self.final_norm.forward(h, rows=ctx.logit_rows, add=pending)
         ops.current_tag = "lm_head"
         return linear.matmul(xn, self.head, self.rt)
+
+    def _write_stream(self, h, pending, out) -> None:
+        """Makes the add that is left and stores the stream as it then stands in `out` [T, D] (operand dtype), in one pass if the
+        add passes a norm that can."""
+        if isinstance(pending, PostNormed) and pending.norm.fuses_mixture:
+            pending.norm.add_normed(h, pending.y, weighted=pending.weighted, raw=out)
+            return
+        if pending is not None:
+            pending.apply(h)
+        ops.layernorm(h, None, None, 0.0, self.rt.dtype, raw=out)

@@ -123,9 +123,11 @@ _ll = ctypes.c_longlong
 
 
 # --------------------------------------------------------------------------- elementwise
-def embed(tokens: torch.Tensor, table: torch.Tensor, out: Optional[torch.Tensor] = None, fed: Optional[torch.Tensor] = None) -> torch.Tensor:
-    """h[t] = float32(table[tokens[t]]).  With `fed` (int32 on the device), a token id -(i + 1)
-    stands for fed[i]: a token the step before has sampled and the host has not read yet."""
+def embed(tokens: torch.Tensor, table: torch.Tensor, out: Optional[torch.Tensor] = None, fed: Optional[torch.Tensor] = None,
+          scale: float = 1.0, copy: Optional[torch.Tensor] = None) -> torch.Tensor:
+    """h[t] = float32(table[tokens[t]]) * scale.  With `fed` (int32 on the device), a token id -(i + 1)
+    stands for fed[i]: a token the step before has sampled and the host has not read yet.  copy: [T, n D] (rows may lie
+    apart, in the table's dtype) that takes the same rows n times side by side."""
     T = tokens.numel()
     V, D = table.shape
     _need(tokens, "tokens", torch.int32)
@@ -135,8 +137,11 @@ def embed(tokens: torch.Tensor, table: torch.Tensor, out: Optional[torch.Tensor]
     if out is None:
         out = torch.empty((T, D), dtype=torch.float32, device=table.device)
     _need(out, "out", torch.float32, (T, D))
+    if copy is not None and (copy.dtype != table.dtype or copy.shape[0] != T or copy.shape[1] % D or copy.stride(1) != 1 or not copy.is_cuda):
+        raise KernelError("embed: the second output does not match the table")
     _call("q6k_embed", _ptr(tokens), _ptr(table), _ptr(out), _i(T), _i(D), _i(V), _i(dtype_code(table.dtype)), _ptr(fed),
-          _i(fed.numel() if fed is not None else 0), _stream())
+          _i(fed.numel() if fed is not None else 0), _f(scale), _ptr(copy), _ll(copy.stride(0) if copy is not None else 0),
+          _i(copy.shape[1] // D if copy is not None else 0), _stream())
     return out
 
 
@@ -882,7 +887,8 @@ def gemm_tc_pairs(a: torch.Tensor, w: torch.Tensor, pair_expert: torch.Tensor, p
                   order: Optional[torch.Tensor] = None, pairs_are_old: bool = False, act: Optional[str] = None) -> torch.Tensor:
     """Expert products of a decode step without a permutation: pair y (= token * slots + slot)
     multiplies row y // pair_div of `a` with expert pair_expert[y]; output row y.  With w2 the
-    SwiGLU epilogue (bfloat16 output), else FP32.  pairs_are_old: the caller's word that
+    SwiGLU epilogue (bfloat16 output), else FP32.  A pair whose expert number is beyond the last matrix is skipped (its
+    output row is left as it is).  pairs_are_old: the caller's word that
     pair_expert and order were not made by the kernel launched just before this one; the kernel
     then fetches its first weights while that kernel still runs."""
     if not tc_supported(a, w) or w.dim() != 3:
@@ -933,11 +939,13 @@ def moe_permute(sel_e: torch.Tensor, E: int):
     return offsets, pair_row, row_token
 
 
-def moe_plan(sel_e: torch.Tensor, E: int, bm: int, x: Optional[torch.Tensor] = None):
+def moe_plan(sel_e: torch.Tensor, E: int, bm: int, x: Optional[torch.Tensor] = None, live: Optional[int] = None):
     """The permutation of `moe_permute` and the row tiles of `tile_list(offsets, pairs, bm)` in three
     launches instead of four: (offsets, pair_row, row_token, (offsets, tile_group, tile_row0, num_tiles)).
     With x [T, D] (rows of a multiple of 16 bytes) the last launch also copies each pair's input
-    row into its place, and the gathered rows [pairs, D] are returned as a fifth value."""
+    row into its place, and the gathered rows [pairs, D] are returned as a fifth value.  live: only the
+    first `live` experts have matrices; the pairs of the others come last and get no tiles and no copies."""
+    live = E if live is None else int(live)
     _need(sel_e, "sel_e", torch.int32)
     T, k = sel_e.shape
     pairs = T * k
@@ -948,7 +956,7 @@ def moe_plan(sel_e: torch.Tensor, E: int, bm: int, x: Optional[torch.Tensor] = N
     offsets = torch.empty(E + 1, dtype=torch.int32, device=dev)
     pair_row = torch.empty((T, k), dtype=torch.int32, device=dev)
     row_token = torch.empty(pairs, dtype=torch.int32, device=dev)
-    max_tiles = pairs // bm + min(pairs, E)          # full tiles plus at most one ragged tile per non-empty group
+    max_tiles = pairs // bm + min(pairs, live)       # full tiles plus at most one ragged tile per non-empty group
     tile_group = torch.empty(max_tiles, dtype=torch.int32, device=dev)
     tile_row0 = torch.empty(max_tiles, dtype=torch.int32, device=dev)
     num_tiles = torch.empty(1, dtype=torch.int32, device=dev)
@@ -961,7 +969,7 @@ def moe_plan(sel_e: torch.Tensor, E: int, bm: int, x: Optional[torch.Tensor] = N
         if row_bytes % 16:
             raise KernelError(f"moe_plan: rows of {row_bytes} bytes cannot be gathered 16 bytes at a time")
         gathered = torch.empty((pairs, x.shape[1]), dtype=x.dtype, device=dev)
-    _call("q6k_moe_plan", _ptr(sel_e), _i(pairs), _i(k), _i(E), _ptr(scratch), _ptr(offsets), _ptr(pair_row), _ptr(row_token), _i(bm),
+    _call("q6k_moe_plan", _ptr(sel_e), _i(pairs), _i(k), _i(E), _i(live), _ptr(scratch), _ptr(offsets), _ptr(pair_row), _ptr(row_token), _i(bm),
           _ptr(tile_group), _ptr(tile_row0), _ptr(num_tiles), _i(max_tiles), _ptr(x), _ptr(gathered), _i(row_bytes), _stream())
     plan = (offsets, pair_row, row_token, (offsets, tile_group, tile_row0, num_tiles))
     return plan if x is None else plan + (gathered,)
@@ -1030,38 +1038,71 @@ def topk_pool(logits: torch.Tensor, k: int):
 
 # --------------------------------------------------------------------------- layer norm, selective scan, flexible attention
 def layernorm(h: torch.Tensor, w: Optional[torch.Tensor], b: Optional[torch.Tensor], eps: float, out_dtype: torch.dtype,
-              rows: Optional[torch.Tensor] = None, after=None, extra: Optional[torch.Tensor] = None) -> Optional[torch.Tensor]:
+              rows: Optional[torch.Tensor] = None, after=None, extra: Optional[torch.Tensor] = None, mixture=None, replace=None,
+              raw: Optional[torch.Tensor] = None) -> Optional[torch.Tensor]:
     """Layer norm with weight and bias on the FP32 stream h [T, D], up to three steps in one pass over each row:
-    after = (y, wa, ba): h += LN(y; wa, ba) first (y FP32 [T, D] or [slices, T, D] partial sums added in order);
-    extra (FP32 like h): h += extra next; w, b: the result LN(h; w, b) in out_dtype (None: no result, h is only
-    updated).  rows: int32 row numbers to normalise (without after and extra)."""
+    after = (y, wa, ba): h += LN(u; wa, ba) first (y FP32 [T, D] or [slices, T, D] partial sums added in order, or None), or
+    replace = (y, vec): h = u + vec (vec FP32 [D] or None); extra (FP32 like h): h += extra next; w, b: the result LN(h; w, b)
+    in out_dtype (None: no result, h is only updated), or raw: a [T, D] buffer in out_dtype (rows may lie apart) that takes the
+    stream as it then stands.  u is y, or with mixture = (py, pair_row, pw, x, xw, gate), each but py optional,
+    gate[t] * y[t] + sum_s pw[t, s] * py[row] (rows as in `combine`; a row of weight zero is not read) + xw[t] * x[t] (x [T, D] in
+    out_dtype).  rows: int32 row numbers whose result is wanted; h then stays as it is."""
     _need(h, "h", torch.float32)
     T, D = h.shape
     R = T if rows is None else rows.numel()
-    y = wa = ba = None
+    y = wa = ba = vec = None
     splits, stride = 1, 0
+    if after is not None and replace is not None:
+        raise KernelError("layernorm: the stream is added to or replaced, not both")
     if after is not None:
         y, wa, ba = after
-        _need(y, "y", torch.float32)
         _need(wa, "wa", torch.float32, (D,))
         _need(ba, "ba", torch.float32, (D,))
+    if replace is not None:
+        y, vec = replace
+        if vec is not None:
+            _need(vec, "vec", torch.float32, (D,))
+    if y is not None:
+        _need(y, "y", torch.float32)
         if y.dim() == 3:
             splits, stride = y.shape[0], y.shape[1] * y.shape[2]
         if tuple(y.shape[-2:]) != (T, D):
             raise KernelError("layernorm: the sublayer's result does not match h")
+    py = pair_row = pw = x = xw = gate = None
+    S = 0
+    if mixture is not None:
+        py, pair_row, pw, x, xw, gate = mixture
+        if after is None and replace is None:
+            raise KernelError("layernorm: routed rows without the norm they pass")
+        if py is not None:
+            _need(py, "routed rows", torch.float32)
+            _need(pw, "weights", torch.float32)
+            S = pw.shape[1]
+            if pair_row is not None:
+                _need(pair_row, "pair_row", torch.int32)
+            if pw.shape[0] != T or py.shape[1] != D or py.shape[0] < T * S or (pair_row is not None and pair_row.numel() != T * S):
+                raise KernelError("layernorm: the routed rows do not match h")
+        if x is not None:
+            _need(x, "x", out_dtype, (T, D))
+            _need(xw, "xw", torch.float32, (T,))
+        if gate is not None:
+            _need(gate, "gate", torch.float32, (T,))
     if extra is not None:
         _need(extra, "extra", torch.float32, (T, D))
     if rows is not None:
         _need(rows, "rows", torch.int32)
-        if after is not None or extra is not None:
-            raise KernelError("layernorm: picked rows are only normalised")
-    out = None
+    out, ldo = None, D
     if w is not None:
         _need(w, "w", torch.float32, (D,))
         _need(b, "b", torch.float32, (D,))
         out = torch.empty((R, D), dtype=out_dtype, device=h.device)
-    _call("q6k_layernorm", _ptr(h), _ptr(y), _i(splits), _ll(stride), _ptr(wa), _ptr(ba), _ptr(extra), _ptr(w), _ptr(b), _ptr(rows),
-          _ptr(out), _i(R), _i(D), _f(eps), _i(dtype_code(out_dtype)), _stream())
+    elif raw is not None:
+        if raw.dtype != out_dtype or tuple(raw.shape) != (R, D) or raw.stride(1) != 1 or not raw.is_cuda:
+            raise KernelError(f"layernorm: the buffer for the stream must be [{R}, {D}] in {out_dtype}")
+        out, ldo = raw, raw.stride(0)
+    _call("q6k_layernorm", _ptr(h), _ptr(y), _i(splits), _ll(stride), _ptr(gate), _ptr(py), _ptr(pair_row), _ptr(pw), _i(S), _ptr(x), _ptr(xw),
+          _ptr(wa), _ptr(ba), _i(1 if replace is not None else 0), _ptr(vec), _ptr(extra), _ptr(w), _ptr(b), _ptr(rows), _ptr(out), _ll(ldo), _i(R), _i(D),
+          _f(eps), _i(dtype_code(out_dtype)), _stream())
     return out
 
 
@@ -1470,23 +1511,34 @@ def activate(x: torch.Tensor, I: int, gated: bool, act: str, out_dtype: torch.dt
     return out
 
 
-def route_biased(logits: torch.Tensor, k: int, bias: Optional[torch.Tensor], scale: float, renorm: bool = True, groups=None, power: int = 1):
-    """(sel_e int32 [T, k], sel_w float32 [T, k]): per row the k experts with the largest sigmoid(logit) + bias (ties to the
-    lower index); weights sigmoid(logit) / (their sum + 1e-20) * scale, or sigmoid(logit) * scale without renorm.
+def route_biased(logits: torch.Tensor, k: int, bias: Optional[torch.Tensor], scale: float, renorm: bool = True, groups=None, power: int = 1,
+                 scoring: str = "sigmoid", group_worth: str = "two", experts: Optional[int] = None, identity: int = 0, gate: bool = False):
+    """(sel_e int32 [T, k], sel_w float32 [T, k]): per row the k experts with the largest score + bias (ties to the
+    lower index), a score being sigmoid(logit), or softmax over all experts' logits; weights score / (their sum + 1e-20) * scale,
+    or score * scale without renorm.
     groups = (count, keep): the experts form `count` equal groups of neighbours, a group's worth is the sum of its two
-    largest choice values, and only experts of the `keep` groups of most worth can be chosen.
-    power = 2: the weights leave squared.  logits: [T, E] or [slices, T, E] partial sums."""
+    largest choice values (group_worth "two") or its largest one ("best"), and only experts of the `keep` groups of most worth
+    can be chosen.  power = 2: the weights leave squared.  logits: [T, N] or [slices, T, N] partial sums; the first `experts`
+    columns (default all) are the experts'.  identity: the last `identity` of the experts answer their input: their weights
+    leave as zero in sel_w, and the row's sum of them is a third result, float32 [T].  gate: sigmoid of column
+    `experts` is one more result, float32 [T]."""
     count, keep = groups if groups is not None else (1, 1)
     _need(logits, "logits", torch.float32)
     slices = logits.shape[0] if logits.dim() == 3 else 1
-    T, E = logits.shape[-2:]
+    T, N = logits.shape[-2:]
+    E = N if experts is None else int(experts)
+    if scoring not in ("sigmoid", "softmax") or group_worth not in ("two", "best"):
+        raise KernelError(f"route_biased: unknown scoring {scoring!r} or worth of a group {group_worth!r}")
     if bias is not None:
         _need(bias, "bias", torch.float32, (E,))
     sel_e = torch.empty((T, k), dtype=torch.int32, device=logits.device)
     sel_w = torch.empty((T, k), dtype=torch.float32, device=logits.device)
-    _call("q6k_route_biased", _ptr(logits), _i(slices), _ptr(bias), _f(scale), _i(T), _i(E), _i(k), _ptr(sel_e), _ptr(sel_w),
-          _i(1 if renorm else 0), _i(count), _i(keep), _i(power), _stream())
-    return sel_e, sel_w
+    id_w = torch.empty(T, dtype=torch.float32, device=logits.device) if identity else None
+    gates = torch.empty(T, dtype=torch.float32, device=logits.device) if gate else None
+    _call("q6k_route_biased", _ptr(logits), _i(slices), _i(N), _ptr(bias), _f(scale), _i(T), _i(E), _i(k), _ptr(sel_e), _ptr(sel_w),
+          _i(1 if renorm else 0), _i(count), _i(keep), _i(power), _i(1 if scoring == "softmax" else 0), _i(1 if group_worth == "best" else 0), _i(identity),
+          _ptr(id_w), _ptr(gates), _stream())
+    return (sel_e, sel_w) + ((id_w,) if identity else ()) + ((gates,) if gate else ())
 
 
 # --------------------------------------------------------------------------- sublayers whose results pass a norm before the stream

@@ -21,6 +21,7 @@ under a name with the matching `register_*`; a spec.PartSpec(kind=name, params=.
   FeedForward     tensors(); bind(); forward(xn [T, D], ctx, out_f32 [T, D]) adds its result into `out`
   Block           built from (norm1, mixer, norm2, ffn); forward(h, ctx, cache, state)
   Connection      tensors(); bind(); what ties a sublayer to a residual of several streams (base.Streams), in arrangements that have one
+  PassEntry       tensors(); bind(); what happens to the stream before each pass over a repeated span of layers
   EmbedAdd        tensors(); bind(); state_shape() as a mixer's; forward(h_f32 [T, D], ctx, state) adds into h in place
 """
 from __future__ import annotations
@@ -106,6 +107,40 @@ class WeightedRows:
     def apply(self, h: torch.Tensor) -> None:
         from .. import ops
         ops.combine(self.y, self.pair_row, self.weights, h)
+
+
+@dataclass
+class Mixture(WeightedRows):
+    """A WeightedRows with what else a routed feed-forward may add: experts that answer their input (x_weights[t] * x[t]; their
+    entries in `weights` are zero and their rows of y are never read), and a number per token that multiplies what stands
+    beside the rows (the shared expert's result).  For norms that say so (Norm.fuses_mixture) and blocks that hand it to them
+    (StepContext.takes_mixture)."""
+    x: Optional[torch.Tensor] = None          # [T, D] in the operand dtype
+    x_weights: Optional[torch.Tensor] = None  # FP32 [T]
+    gate: Optional[torch.Tensor] = None       # FP32 [T]
+
+    def made(self, beside: Optional[torch.Tensor]) -> torch.Tensor:
+        """gate * beside + the weighted rows + x_weights * x, FP32 [T, D] (beside: FP32 [T, D], split-K slices or None)."""
+        from .. import ops
+        out = torch.empty((self.weights.shape[0], self.y.shape[1]), dtype=torch.float32, device=self.y.device)
+        dtype = self.x.dtype if self.x is not None else torch.float32
+        ops.layernorm(out, None, None, 0.0, dtype, replace=(beside, None), mixture=(self.y, self.pair_row, self.weights, self.x, self.x_weights, self.gate))
+        return out
+
+    def apply(self, h: torch.Tensor) -> None:
+        h += self.made(None)
+
+
+@dataclass
+class Replaced:
+    """A change of the stream that has not been made yet: h <- y + vec (y FP32 [T, D], or [slices, T, D] partial sums to be
+    added in order; vec FP32 [D])."""
+    y: torch.Tensor
+    vec: Optional[torch.Tensor] = None
+
+    def apply(self, h: torch.Tensor) -> None:
+        from .. import ops
+        ops.layernorm(h, None, None, 0.0, torch.float32, replace=(self.y, self.vec))
 
 
 @dataclass
@@ -209,6 +244,8 @@ class Tap:
 class Norm(Part):
     fuses_weighted_rows = False           # forward(..., add=WeightedRows) is understood
     fuses_post_normed = False             # forward(..., add=PostNormed) is understood
+    fuses_picked_rows = False             # ... also together with rows: the add is then made for the picked rows only
+    fuses_mixture = False                 # add_normed and PostNormed may come with a Mixture
 
     def add_normed(self, h: torch.Tensor, y: torch.Tensor) -> None:
         """h += this norm of y (y FP32 [T, D] or [slices, T, D] partial sums), in place."""
@@ -263,6 +300,18 @@ class EmbedAdd(Part):
         raise NotImplementedError
 
 
+class PassEntry(Part):
+    """What happens to the stream right before each pass over a span of layers that runs several times: open(h, operand, n)
+    returns what is left to the span's first norm (a Replaced, or None).  operand [T, operand_width()] is in the operand
+    dtype: its last D columns hold the embedding output, its first D the stream as it stands."""
+
+    def operand_width(self) -> int:
+        raise NotImplementedError
+
+    def open(self, h: torch.Tensor, operand: torch.Tensor, n: int):
+        raise NotImplementedError
+
+
 class Connection(Part):
     """What ties a sublayer to a residual of several streams."""
 
@@ -305,6 +354,7 @@ FEED_FORWARDS: Dict[str, type] = {}
 BLOCKS: Dict[str, type] = {}
 EMBED_ADDS: Dict[str, type] = {}
 CONNECTIONS: Dict[str, type] = {}
+PASS_ENTRIES: Dict[str, type] = {}
 
 
 def _register(table: Dict[str, type], what: str):
@@ -323,6 +373,7 @@ register_feed_forward = _register(FEED_FORWARDS, "feed-forward")
 register_block = _register(BLOCKS, "block")
 register_embed_add = _register(EMBED_ADDS, "embedding add")
 register_connection = _register(CONNECTIONS, "connection")
+register_pass_entry = _register(PASS_ENTRIES, "entry of a pass")
 
 
 def make_part(table: Dict[str, type], what: str, spec: PartSpec, **extra):

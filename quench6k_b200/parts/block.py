@@ -42,6 +42,11 @@ class SandwichBlock(Block):
             return PostNormed(y, self.norm1b)
         ops.current_tag = "norm.ffn"
         xn = self.norm2.forward(h, add=PostNormed(y, self.norm1b))
+        if getattr(self.ffn, "defers_add", False):
+            ctx.takes_mixture = self.norm2b.fuses_mixture     # the norm sums what the experts leave unsummed
+            y, rows = self.ffn.compute(xn, ctx)
+            ctx.takes_mixture = False
+            return PostNormed(y, self.norm2b, rows)
         return PostNormed(self.ffn.compute(xn, ctx), self.norm2b)
 
 

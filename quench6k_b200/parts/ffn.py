@@ -15,7 +15,7 @@ import torch
 from .. import ops
 from ..spec import TensorSpec
 from . import linear
-from .base import FeedForward, WeightedRows, register_feed_forward, to_f32, to_operand
+from .base import FeedForward, Mixture, WeightedRows, register_feed_forward, to_f32, to_operand
 
 
 _DEGREE = {"relu2": 2}             # activations f with f(w z) = w^n f(z) for w >= 0: their n
@@ -74,12 +74,15 @@ class RoutedExperts(FeedForward):
     def __init__(self, hidden_size: int, num_experts: int, top_k: int, intermediate_size: int, scoring: str = "softmax",
                  renormalize: bool = True, shared_intermediate_size: int = 0, gated: bool = True, act: str = "silu",
                  correction: bool = False, route_scale: float = 1.0, names=None, shared_act=None, shared_prefix: str = "shared_experts.",
-                 shared_names=None, groups=None, weights_on_input: bool = False):
+                 shared_names=None, groups=None, weights_on_input: bool = False, group_worth: str = "two", identity: int = 0,
+                 shared_gate: bool = False):
         """gated: an expert is down(act(gate x) * (up x)); else down(act(up x)).  correction: a stored vector added to the
         scores for the choice of the experts only (the weights use the scores without it); route_scale multiplies the
         weights.  groups = (count, keep): the experts form `count` equal groups of neighbours, and only experts of the `keep`
-        groups whose two largest choice values add up to most can be chosen.  All three belong to sigmoid scoring (with
-        renormalised weights, or with the plain scores as weights).  act may be a gate with its constant, such as
+        groups of most worth can be chosen, a group's worth being its two largest choice values added (group_worth "two") or its
+        largest one ("best").  identity: this many further experts, numbered after the others and known to the router, the
+        correction and the groups, answer their input and have no tensors.  shared_gate: the shared expert's result is
+        multiplied by sigmoid of one more projection of the input, one number per token.  act may be a gate with its constant, such as
         ("clamped", limit) (gated experts only).  The shared expert has the experts' form with an activation (shared_act,
         default the experts'), a tensor prefix and tensor names of its own.  weights_on_input: a weight multiplies its expert's
         INPUT.  An expert without a gate whose activation is homogeneous of degree n answers w x with w^n times its answer to x
@@ -89,41 +92,50 @@ class RoutedExperts(FeedForward):
             raise ValueError(f"the gate {act[0]!r} belongs to gated experts")
         self.gated, self.act, self.has_correction, self.route_scale = bool(gated), act, bool(correction), float(route_scale)
         self.groups = (int(groups[0]), int(groups[1])) if groups is not None and int(groups[0]) > 1 else None
-        if self.groups is not None and (num_experts % self.groups[0] or not 0 < self.groups[1] <= self.groups[0]
-                                        or top_k > self.groups[1] * (num_experts // self.groups[0])):
-            raise ValueError(f"{num_experts} experts in {self.groups[0]} groups of which {self.groups[1]} are kept, {top_k} chosen")
+        self.group_worth, self.identity, self.shared_gate = group_worth, int(identity), bool(shared_gate)
+        total = num_experts + self.identity                # what the router chooses from
+        if self.identity < 0 or group_worth not in ("two", "best"):
+            raise ValueError(f"{identity} experts that answer their input, worth of a group {group_worth!r}")
+        if self.shared_gate and shared_intermediate_size <= 0:
+            raise ValueError("a gate on the shared expert needs a shared expert")
+        if self.groups is not None and (total % self.groups[0] or not 0 < self.groups[1] <= self.groups[0]
+                                        or top_k > self.groups[1] * (total // self.groups[0])):
+            raise ValueError(f"{total} experts in {self.groups[0]} groups of which {self.groups[1]} are kept, {top_k} chosen")
         self.weight_power = 1
         if weights_on_input:
             if gated or act not in _DEGREE or scoring != "sigmoid":
                 raise ValueError(f"weights on the experts' input: experts without a gate, sigmoid scores and an activation of {', '.join(_DEGREE)}")
             self.weight_power = _DEGREE[act]
-        self.own_router = self.has_correction or self.route_scale != 1.0 or self.groups is not None or self.weight_power != 1
-        if self.own_router and scoring != "sigmoid":
-            raise ValueError("a correction of the choice, groups of experts and a scale of the weights go with sigmoid scores")
+        self.own_router = (self.has_correction or self.route_scale != 1.0 or self.groups is not None or self.weight_power != 1 or self.identity > 0
+                           or self.shared_gate)
         self.names = {"router": "gate.weight", "gate": "experts.gate_proj.weight", "up": "experts.up_proj.weight",
-                      "down": "experts.down_proj.weight", "correction": "gate.correction", **(names or {})}
+                      "down": "experts.down_proj.weight", "correction": "gate.correction", "shared_gate": "shared_gate.weight", **(names or {})}
         if scoring not in ("softmax", "sigmoid"):
             raise ValueError(f"unknown router scoring {scoring!r}")
-        if not 0 < top_k <= num_experts:
-            raise ValueError(f"top_k {top_k} outside 1..{num_experts}")
+        if not 0 < top_k <= total:
+            raise ValueError(f"top_k {top_k} outside 1..{total}")
+        self.total = total
+        self.ng = -(-(total + 1) // 8) * 8 - total if self.shared_gate else 0      # rows the gate adds to the router product, with padding
         self.D, self.E, self.k, self.I = hidden_size, num_experts, top_k, intermediate_size
         self.scoring, self.renorm = scoring, bool(renormalize)
         self.shared_prefix = shared_prefix
         self.shared = (DenseSwiGLU(hidden_size, shared_intermediate_size, names=shared_names, act=shared_act if shared_act is not None else act)
                        if shared_intermediate_size > 0 else None)
-        self.always_defers = self.shared is None      # forward(defer=True) never touches `out`
+        self.always_defers = self.shared is None and not self.identity      # forward(defer=True) never touches `out`
         self.pair_tokens = 16                         # steps of at most this many tokens run the experts pair by pair
         self.routing_tap = None               # a parts.base.Tap: every forward records each row's chosen experts [T, k]
                                               # ("experts") and its router logits [T, E] ("router_logits") there
 
     def tensors(self):
         E, I, D, n = self.E, self.I, self.D, self.names
-        out = [TensorSpec(n["router"], (E, D))]
+        out = [TensorSpec(n["router"], (self.total, D))]
         if self.gated:
             out.append(TensorSpec(n["gate"], (E, I, D)))
         out += [TensorSpec(n["up"], (E, I, D)), TensorSpec(n["down"], (E, D, I))]
         if self.has_correction:
-            out.append(TensorSpec(n["correction"], (E,), "f32", ("normal", 0.1)))
+            out.append(TensorSpec(n["correction"], (self.total,), "f32", ("normal", 0.1)))
+        if self.shared_gate:
+            out.append(TensorSpec(n["shared_gate"], (1, D)))
         if self.shared is not None:
             out += [TensorSpec(self.shared_prefix + t.name, t.shape, t.role, t.init) for t in self.shared.tensors()]
         return out
@@ -131,7 +143,12 @@ class RoutedExperts(FeedForward):
     def bind(self, get, rt):
         self.rt = rt
         n = self.names
-        self.w_router = to_operand(get(n["router"]), rt)
+        if self.shared_gate:                               # the gate's row rides in the router product
+            self.w_router = torch.zeros((self.total + self.ng, self.D), dtype=rt.dtype, device=rt.device)
+            self.w_router[:self.total].copy_(get(n["router"]))
+            self.w_router[self.total:self.total + 1].copy_(get(n["shared_gate"]))
+        else:
+            self.w_router = to_operand(get(n["router"]), rt)
         self.w_up = to_operand(get(n["up"]), rt)
         self.w_gate = to_operand(get(n["gate"]), rt) if self.gated else self.w_up      # ungated: the first (only) product's weights
         self.w_down = to_operand(get(n["down"]), rt)
@@ -148,19 +165,38 @@ class RoutedExperts(FeedForward):
                 total += logits[s]
             logits = total
         self.routing_tap.record("experts", ctx.position, sel_e)
-        self.routing_tap.record("router_logits", ctx.position, logits)
+        self.routing_tap.record("router_logits", ctx.position, logits[:, :self.total])
+
+    def _rows(self, y, sel_w, pair_row, xn, more):
+        """The experts' results unsummed; more: what the router said of the experts that answer their input and of the gate."""
+        if not (self.identity or self.shared_gate):
+            return WeightedRows(y, sel_w, pair_row)
+        more = list(more)
+        id_w = more.pop(0) if self.identity else None
+        return Mixture(y, sel_w, pair_row, x=xn if self.identity else None, x_weights=id_w, gate=more.pop(0) if self.shared_gate else None)
 
     def compute(self, xn, ctx):
         """(the shared expert's result FP32 [T, D] or split-K slices of it, or None; the routed experts' results unsummed,
-        a WeightedRows): for a block whose norm takes the sum before the stream does."""
+        a WeightedRows): for a block whose norm takes the sum before the stream does.  Experts that answer their input and
+        a gate on the shared expert make it a Mixture for blocks that take one; for the others the sum is made here."""
         rows = self.forward(xn, ctx, None, defer=True, routed_only=True)
-        return (self.shared.compute(xn, ctx) if self.shared is not None else None), rows
+        both = self.shared.compute(xn, ctx) if self.shared is not None else None
+        if isinstance(rows, Mixture) and not ctx.takes_mixture:
+            ops.current_tag = "experts.combine"
+            return rows.made(both), None
+        return both, rows
 
     def forward(self, xn, ctx, out, defer=False, routed_only=False):
         """Adds the experts' weighted results into `out`; with defer=True and no shared expert it
         returns them unsummed (WeightedRows) for the next norm to add.  routed_only: the shared expert is the caller's."""
         rt = self.rt
         T = xn.shape[0]
+        if (self.identity or self.shared_gate) and not routed_only:
+            y, rows = self.compute(xn, ctx)
+            if rows is not None:
+                y = rows.made(y)
+            out += y
+            return None
         pairs = T * self.k
         defer = defer and (self.shared is None or routed_only)
         if (self.gated and self.act == "silu" and not self.own_router and rt.tensor_cores and not rt.is_fp32 and ops.router_small_supported(T, self.E, self.D, self.k)
@@ -190,9 +226,12 @@ class RoutedExperts(FeedForward):
         ops.current_tag = "experts.router"
         logits = linear.matmul(xn, self.w_router, rt, partials_ok=True)    # FP32 [T, E], or split-K slices of it that route() sums
         if self.own_router:
-            sel_e, sel_w = ops.route_biased(logits, self.k, self.correction, self.route_scale, renorm=self.renorm, groups=self.groups, power=self.weight_power)
+            sel_e, sel_w, *more = ops.route_biased(logits, self.k, self.correction, self.route_scale, renorm=self.renorm, groups=self.groups,
+                                                   power=self.weight_power, scoring=self.scoring, group_worth=self.group_worth, experts=self.total,
+                                                   identity=self.identity, gate=self.shared_gate)
         else:
             sel_e, sel_w = ops.route(logits, self.k, self.scoring, self.renorm)
+            more = ()
         if self.routing_tap is not None:
             self._tap(ctx, sel_e, logits)
         if (T <= self.pair_tokens and defer and rt.tensor_cores and not rt.is_fp32 and ops.tc_supported(xn, self.w_up) and self.I % 8 == 0):
@@ -202,9 +241,9 @@ class RoutedExperts(FeedForward):
             act = self.act if not self.gated or self.act != "silu" else None
             first = ops.gemm_tc_pairs(xn, self.w_gate, sel_e, self.k, w2=self.w_up if self.gated else None, act=act)     # [pairs, I]
             ops.current_tag = "experts.down"
-            return WeightedRows(ops.gemm_tc_pairs(first, self.w_down, sel_e, 1, pairs_are_old=True), sel_w)
+            return self._rows(ops.gemm_tc_pairs(first, self.w_down, sel_e, 1, pairs_are_old=True), sel_w, None, xn, more)
         ops.current_tag = "experts.permute"
-        plan = linear.group_plan(xn, self.w_gate, sel_e, rt)             # permutation by expert, row tiles, gathered rows
+        plan = linear.group_plan(xn, self.w_gate, sel_e, rt, without=self.identity)             # permutation by expert, row tiles, gathered rows
         ops.current_tag = "experts.gate_up"
         if self.gated:
             act = linear.grouped_swiglu(xn, plan, self.w_gate, self.w_up, rt, act=None if self.act == "silu" else self.act)   # [pairs, I]
@@ -213,7 +252,7 @@ class RoutedExperts(FeedForward):
         ops.current_tag = "experts.down"
         y = linear.grouped_matmul(act, plan, self.w_down, rt)                                     # FP32 [pairs, D]
         if defer:
-            return WeightedRows(y, sel_w, plan.pair_row)
+            return self._rows(y, sel_w, plan.pair_row, xn, more)
         ops.current_tag = "experts.combine"
         ops.combine(y, plan.pair_row, sel_w, out)
         if self.shared is not None:

@@ -53,7 +53,9 @@ class GroupPlan:
     """The permutation of a step's (token, slot) pairs by expert and the row tiles of the experts'
     groups, for whichever kernel runs them; on the tensor-core path also the gathered input rows."""
 
-    def __init__(self, a: torch.Tensor, sel_e: torch.Tensor, num_groups: int, rt, tc: bool):
+    def __init__(self, a: torch.Tensor, sel_e: torch.Tensor, num_groups: int, rt, tc: bool, live: int):
+        """num_groups: expert numbers there are; live: those that have matrices (the pairs of the others get no tiles)."""
+        self.live = live
         self.pairs, self.tc, self.xs = sel_e.numel(), tc, None
         if tc:
             avg = max(1, self.pairs // max(1, num_groups))
@@ -63,16 +65,17 @@ class GroupPlan:
             # permutation, tile list and the gathered input rows in three launches (the last one, a block per pair,
             # finishes the pair's rank and copies its row)
             if a.shape[1] * a.element_size() % 16 == 0:
-                self.offsets, self.pair_row, self.row_token, self.tiles, self.xs = ops.moe_plan(sel_e, num_groups, self.bt, a)
+                self.offsets, self.pair_row, self.row_token, self.tiles, self.xs = ops.moe_plan(sel_e, num_groups, self.bt, a, live=live)
             else:
-                self.offsets, self.pair_row, self.row_token, self.tiles = ops.moe_plan(sel_e, num_groups, self.bt)
+                self.offsets, self.pair_row, self.row_token, self.tiles = ops.moe_plan(sel_e, num_groups, self.bt, live=live)
                 self.xs = ops.gather_rows(a, self.row_token)
         else:
-            self.offsets, self.pair_row, self.row_token, self.tiles = ops.moe_plan(sel_e, num_groups, ops.simt_tile_rows())
+            self.offsets, self.pair_row, self.row_token, self.tiles = ops.moe_plan(sel_e, num_groups, ops.simt_tile_rows(), live=live)
 
 
-def group_plan(a: torch.Tensor, w: torch.Tensor, sel_e: torch.Tensor, rt) -> GroupPlan:
-    return GroupPlan(a, sel_e, w.shape[0], rt, _tc(a, w, rt) and a.is_contiguous())
+def group_plan(a: torch.Tensor, w: torch.Tensor, sel_e: torch.Tensor, rt, without: int = 0) -> GroupPlan:
+    """without: expert numbers beyond the last matrix of w, whose pairs take part in no product."""
+    return GroupPlan(a, sel_e, w.shape[0] + without, rt, _tc(a, w, rt) and a.is_contiguous(), w.shape[0])
 
 
 def grouped_swiglu(a: torch.Tensor, plan: GroupPlan, w_gate: torch.Tensor, w_up: torch.Tensor, rt, act=None) -> torch.Tensor:
@@ -95,7 +98,7 @@ def grouped_matmul(a: torch.Tensor, plan: GroupPlan, w: torch.Tensor, rt) -> tor
     if plan.tc and ops.tc_supported(a, w):
         return ops.gemm_tc(a, w, groups=plan.tiles, bt=plan.bt, rows=plan.pairs)
     if plan.tc:
-        return ops.gemm_simt(a, w, groups=ops.tile_list(plan.tiles[0], plan.pairs, ops.simt_tile_rows()), rows=plan.pairs)
+        return ops.gemm_simt(a, w, groups=ops.tile_list(plan.tiles[0][:plan.live + 1], plan.pairs, ops.simt_tile_rows()), rows=plan.pairs)
     return ops.gemm_simt(a, w, groups=plan.tiles, rows=plan.pairs)
 
 

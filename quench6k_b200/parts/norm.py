@@ -4,7 +4,7 @@ from __future__ import annotations
 
 from .. import ops
 from ..spec import TensorSpec
-from .base import Norm, PostNormed, WeightedRows, register_norm, to_f32
+from .base import Mixture, Norm, PostNormed, Replaced, WeightedRows, register_norm, to_f32
 
 
 @register_norm("rmsnorm")
@@ -52,13 +52,14 @@ class RMSNorm(Norm):
 @register_norm("layernorm")
 class LayerNorm(Norm):
     """out = (x - mean) / sqrt(var + eps) * w + b, the variance being the mean of the squared deviations; FP32.
-    weight_name / bias_name: the tensors' names relative to the norm's prefix (an architecture may call them anything)."""
+    weight_name / bias_name: the tensors' names relative to the norm's prefix (an architecture may call them anything).
+    mult: the result is multiplied by this constant (weight and bias take it when they are bound)."""
     graph_safe = True
-    fuses_post_normed = True
+    fuses_post_normed = fuses_picked_rows = fuses_mixture = True
 
-    def __init__(self, size: int, eps: float, init: str = "ones", weight_name: str = "weight", bias_name: str = "bias"):
+    def __init__(self, size: int, eps: float, init: str = "ones", weight_name: str = "weight", bias_name: str = "bias", mult: float = 1.0):
         self.size, self.eps, self.init = size, float(eps), init
-        self.weight_name, self.bias_name = weight_name, bias_name
+        self.weight_name, self.bias_name, self.mult = weight_name, bias_name, float(mult)
 
     def tensors(self):
         plain = self.init == "ones"
@@ -68,16 +69,31 @@ class LayerNorm(Norm):
     def bind(self, get, rt):
         self.rt = rt
         self.weight, self.bias = to_f32(get(self.weight_name), rt), to_f32(get(self.bias_name), rt)
+        if self.mult != 1.0:
+            self.weight, self.bias = (self.weight * self.mult).contiguous(), (self.bias * self.mult).contiguous()
 
-    def add_normed(self, h, y):
-        ops.layernorm(h, None, None, self.eps, self.rt.dtype, after=(y, self.weight, self.bias))
+    @staticmethod
+    def _mixture(weighted):
+        """A WeightedRows (or Mixture) as ops.layernorm takes it."""
+        if weighted is None:
+            return None
+        more = (weighted.x, weighted.x_weights, weighted.gate) if isinstance(weighted, Mixture) else (None, None, None)
+        return (weighted.y, weighted.pair_row, weighted.weights, *more)
+
+    def add_normed(self, h, y, weighted=None, raw=None):
+        """h += this norm of (y + weighted rows) in place; raw: a [T, D] buffer in the operand dtype that takes the stream as it
+        then stands."""
+        ops.layernorm(h, None, None, self.eps, self.rt.dtype, after=(y, self.weight, self.bias), mixture=self._mixture(weighted), raw=raw)
 
     def forward(self, h, rows=None, add=None, extra=None):
-        """add: a PostNormed of a layer norm (h += its norm of its y, in the same pass), or FP32 to be added as it is;
-        extra: FP32 of h's shape, added after that."""
-        after = None
-        if isinstance(add, PostNormed) and isinstance(add.norm, LayerNorm) and add.norm.eps == self.eps and rows is None:
-            after = (add.y, add.norm.weight, add.norm.bias)
+        """add: a PostNormed of a layer norm (h += its norm of its y, in the same pass), a Replaced (h <- its y + vec, in the
+        same pass), or FP32 to be added as it is; extra: FP32 of h's shape, added after that.  rows: with a PostNormed the
+        picked rows are normed as they would stand and h is left alone (nothing reads it afterwards)."""
+        after = mixture = replace = None
+        if isinstance(add, PostNormed) and isinstance(add.norm, LayerNorm) and add.norm.eps == self.eps:
+            after, mixture = (add.y, add.norm.weight, add.norm.bias), self._mixture(add.weighted)
+        elif isinstance(add, Replaced):
+            replace = (add.y, add.vec)
         elif add is not None:
             if hasattr(add, "apply"):
                 add.apply(h)
@@ -86,4 +102,4 @@ class LayerNorm(Norm):
         if rows is not None and extra is not None:
             h += extra
             extra = None
-        return ops.layernorm(h, self.weight, self.bias, self.eps, self.rt.dtype, rows=rows, after=after, extra=extra)
+        return ops.layernorm(h, self.weight, self.bias, self.eps, self.rt.dtype, rows=rows, after=after, extra=extra, mixture=mixture, replace=replace)

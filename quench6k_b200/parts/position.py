@@ -5,6 +5,8 @@ literal base 10000); "none" leaves q and k as they are (the reference's per-laye
 crates/engine/src/flint.rs:254,408).  An encoding that is no rotation implements `apply`."""
 from __future__ import annotations
 
+import math
+
 import torch
 
 from .base import PositionEncoding, register_position_encoding
@@ -16,9 +18,17 @@ class Rotary(PositionEncoding):
     dimensions of the head rotate (default: all; fewer is partial rotary, the rest pass through).
     pairing: "halves" (d with d + rotary_dim/2, the reference's) or "neighbours" (2i with 2i+1).
     The inverse frequencies are computed in double precision and rounded to float32 once; the
-    angle is the float32 product of position and inverse frequency, as in the reference."""
+    angle is the float32 product of position and inverse frequency, as in the reference.
+    scaling = (factor, low, high, original): by how many turns a pair makes within `original` positions.  Fewer than `low`: it
+    turns `factor` times slower; more than `high`: as it would; between the two the pace is blended linearly in the turns."""
 
-    def __init__(self, head_dim: int, theta: float, rotary_dim: int = 0, pairing: str = "halves"):
+    def __init__(self, head_dim: int, theta: float, rotary_dim: int = 0, pairing: str = "halves", scaling=None):
+        self.scaling = None
+        if scaling is not None:
+            self.scaling = tuple(float(x) for x in scaling)
+            factor, low, high, original = self.scaling
+            if factor <= 0 or original <= 0 or high < low:
+                raise ValueError(f"rotary scaling: factor {factor}, low {low}, high {high}, original {original}")
         self.head_dim, self.theta = head_dim, float(theta)
         self.rotary_dim = int(rotary_dim) or head_dim
         if pairing not in ("halves", "neighbours"):
@@ -31,7 +41,13 @@ class Rotary(PositionEncoding):
     def bind(self, get, rt):
         self.rt = rt
         i = torch.arange(self.rotary_dim // 2, dtype=torch.float64)
-        self.inv_freq = (self.theta ** (-(2.0 * i) / self.rotary_dim)).to(torch.float32).to(rt.device)
+        f = self.theta ** (-(2.0 * i) / self.rotary_dim)
+        if self.scaling is not None:
+            factor, low, high, original = self.scaling
+            turns = original * f / (2.0 * math.pi)
+            keep = ((turns - low) / (high - low)).clamp(0.0, 1.0) if high > low else (turns >= low).to(f.dtype)
+            f = (1.0 - keep) * f / factor + keep * f
+        self.inv_freq = f.to(torch.float32).to(rt.device)
 
     def rotary_table(self):
         return self.inv_freq, self.rotary_dim, self.pairing == "neighbours"

@@ -54,6 +54,12 @@ class ModelSpec:
     # executed positions before which the embedding output is added to the stream again (a span of layers run several
     # times takes its input anew at the start of every pass but the first)
     readd_embedding: Tuple[int, ...] = ()
+    # what happens to the stream right before each pass over a span of layers that runs several times (a key of
+    # parts.PASS_ENTRIES), and the executed positions that open a pass (the first one too); its tensors' names follow the prefix
+    pass_entry: Optional[PartSpec] = None
+    pass_starts: Tuple[int, ...] = ()
+    pass_entry_prefix: str = "model.loop."
+    embed_scale: float = 1.0               # the embedding table's rows enter the stream multiplied by this
     embed_norm: Optional[PartSpec] = None  # a norm applied to the embedding output before the first layer
     embed_norm_prefix: str = "model.embed_norm."
     # a second embedding table (name, columns): the step gathers the tokens' rows of it once, FP32, and layers read their
