@@ -477,7 +477,22 @@ def gunenex_config(size):
     return {"architecture": "Gunenex", "vocab": 32768, "width": D, "streams": 4, "norm": {"eps": 1e-6}, "kv_page_size": 16, "layers": layers}
 
 
-DESIGNS = {"gunenex": (("gunenex", gunenex_config), ("sigusun", sigusun_config), ("kipedra", kipedra_config)),
+def kodatar_config(size):
+    """Kodatar at layer sizes that resemble a real model's: four attention layers inside chunks, each with routed experts (a
+    fifth of what the router knows are identity experts) chosen among the best groups and a gated shared expert; the four run
+    in two passes, each opened by a product over the stream and the embedding output."""
+    D, heads, kv, E, same, top, eff, chunk = {"s": (1024, 8, 2, 32, 8, 4, 512, 1024), "m": (2048, 16, 4, 64, 16, 4, 1024, 2048)}[size]
+    layer = {"type": "attention",
+             "mixer": {"heads": heads, "kv_heads": kv, "dim": 128, "vdim": 128, "scale": 128 ** -0.5, "mask": {"size": chunk},
+                       "rot": {"base": 500000.0, "dims": 128, "scaling": {"factor": 4.0, "low": 1.0, "high": 4.0, "original": 8192}}},
+             "mlp": {"kind": "moe", "expert": {"ff": eff}, "shared": {"ff": eff},
+                     "router": {"experts": E, "identity": same, "top": top, "groups": {"count": 8, "keep": 4}}}}
+    return {"architecture": "Kodatar", "vocab": 32768, "width": D, "norm": {"eps": 1e-6}, "embedding": {"scale": 4.0}, "logit_scale": 0.5,
+            "kv_page_size": 16, "layers": [layer] * 4, "loop": {"start": 0, "stop": 4, "times": 2}}
+
+
+DESIGNS = {"kodatar": (("kodatar", kodatar_config), ("kitodra", kitodra_config), ("pedotar", pedotar_config)),
+           "gunenex": (("gunenex", gunenex_config), ("sigusun", sigusun_config), ("kipedra", kipedra_config)),
            "pedotar": (("pedotar", pedotar_config), ("flint_dense", flint_dense_config)),
            "kitodra": (("kitodra", kitodra_config), ("sigusun", sigusun_config), ("kipedra", kipedra_config)),
            "kipedra": (("kipedra", kipedra_config), ("flint_routed", flint_routed_config)),
@@ -644,9 +659,9 @@ def main():
     ap.add_argument("--profile-ops", action="store_true",
                     help="instead of the benchmark line: where an eager decode step and a prefill step spend their time, launcher by "
                          "launcher (CUDA events around every launch; its own JSON line)")
-    ap.add_argument("--design", default=None, choices=["pedotar", "kipedra", "sigusun", "kitodra", "gunenex"],
+    ap.add_argument("--design", default=None, choices=["pedotar", "kipedra", "sigusun", "kitodra", "gunenex", "kodatar"],
                     help="instead of the benchmark line: prefill and decode throughput of that design beside the closest Flint model "
-                         "(pedotar: dense feed-forwards; kipedra: windows and routed experts; sigusun: beside Kipedra and Pedotar; kitodra: beside Sigusun and Kipedra) at equal layer sizes (--sizes), with each "
+                         "(pedotar: dense feed-forwards; kipedra: windows and routed experts; sigusun: beside Kipedra and Pedotar; kitodra: beside Sigusun and Kipedra; kodatar: beside Kitodra and Pedotar) at equal layer sizes (--sizes), with each "
                          "model's time launcher by launcher (its own JSON line)")
     ap.add_argument("--sizes", default="s,m", help="--design: s (width 1024) and/or m (width 2048)")
     ap.add_argument("--kernel", default=None, choices=["attention_prefill", "gated_delta", "retention", "delta_channel", "time_mix", "hyper_step"],

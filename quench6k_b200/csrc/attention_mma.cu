@@ -46,7 +46,7 @@ struct AttnParams {
     const int* work;                         // [n_work, 8] from attention_plan_kernel: one record per CTA column
     const int* tile_plan;                    // [n_tiles, 4]: first row, tokens, splits, first work item
     int n_work;
-    int max_blocks, page_size, window, Hq, Hkv, G;
+    int max_blocks, page_size, window, chunk, Hq, Hkv, G;
     float scale_log2;
     int early;                               // the plan, the block tables and every key before a tile's first position are older than the
                                              // kernel launched before this one: key tiles may be fetched before the wait for it
@@ -119,16 +119,16 @@ __device__ __forceinline__ int plan_block_sum(int v, int* red) {
 
 __global__ void __launch_bounds__(PLAN_THREADS) attention_plan_kernel(const int* positions, const int* req_of_token,
                                                                        const int* tile_tok0, const int* tile_ntok,
-                                                                       int n_tiles, int window, int n_work, int min_per, int* work,
+                                                                       int n_tiles, int window, int chunk, int n_work, int min_per, int* work,
                                                                        int* tile_plan) {
     pdl_enter();
     __shared__ int red[PLAN_THREADS / 32];
     __shared__ int scan[PLAN_THREADS];
     const int tid = threadIdx.x;
-    const int chunk = (n_tiles + PLAN_THREADS - 1) / PLAN_THREADS, i0 = tid * chunk, i1 = min(n_tiles, i0 + chunk);
+    const int share = (n_tiles + PLAN_THREADS - 1) / PLAN_THREADS, i0 = tid * share, i1 = min(n_tiles, i0 + share);
     auto key_tiles = [&](int i) {
         const int tok0 = tile_tok0[i], first = positions[tok0], last = first + tile_ntok[i] - 1;
-        const int k_lo = window > 0 ? max(0, first - window + 1) : 0;
+        const int k_lo = q6k_first_seen(first, window, chunk);
         return last / KT + 1 - k_lo / KT;
     };
     long long mine = 0;
@@ -246,7 +246,7 @@ __global__ void __launch_bounds__((WIDE ? 8 : 4) * 32 + 32, WIDE ? 1 : 2) attent
     if (tok0 < 0) return;
     const int pos_last = pos_first + ntok - 1;
     const int* bt = p.block_table + (size_t)wa.w * p.max_blocks;
-    const int k_lo = p.window > 0 ? max(0, pos_first - p.window + 1) : 0;        // first key any row of the tile sees
+    const int k_lo = q6k_first_seen(pos_first, p.window, p.chunk);        // first key any row of the tile sees
     const int first_tile = k_lo / KT, end_tile = pos_last / KT + 1;
     const int t_begin = first_tile + part * per, n_mine = max(0, min(end_tile, t_begin + per) - t_begin);
 
@@ -362,7 +362,7 @@ __global__ void __launch_bounds__((WIDE ? 8 : 4) * 32 + 32, WIDE ? 1 : 2) attent
         for (int c = 0; c < 2; ++c) {
             const int tt = (row0 + nb * 8 + 2 * pair + c) / G, pos = pos_first + tt;
             see_to[nb][c] = tt < ntok ? pos : -1;                            // a row past the tile's tokens sees nothing
-            see_from[nb][c] = p.window > 0 ? pos - p.window + 1 : 0;
+            see_from[nb][c] = q6k_first_seen(pos, p.window, p.chunk);
         }
     // Q^T as the first product's B operand: this thread's row is nb*8 + quad, its head dimensions
     // 16 ks + 2 pair + {0, 1} and + 8
@@ -947,12 +947,12 @@ Q6K_API int q6k_attention_status() {
 // 16-byte aligned; n_work >= n_tiles CTAs per KV head share the key tiles, none walking fewer than min_per unless
 // its tile has no more.
 Q6K_API int q6k_attention_plan(const int* positions, const int* req_of_token, const int* tile_tok0, const int* tile_ntok, int n_tiles,
-                               int window, int n_work, int min_per, int* work, int* tile_plan, cudaStream_t st) {
+                               int window, int chunk, int n_work, int min_per, int* work, int* tile_plan, cudaStream_t st) {
     if (n_tiles == 0) return 0;
-    Q6K_REQUIRE(n_work >= n_tiles && window >= 0 && min_per >= 1, "attention_plan: %d work items for %d tiles (window %d, at least %d key tiles each)",
+    Q6K_REQUIRE(n_work >= n_tiles && window >= 0 && chunk >= 0 && min_per >= 1, "attention_plan: %d work items for %d tiles (window %d, at least %d key tiles each)",
                 n_work, n_tiles, window, min_per);
     Q6K_REQUIRE(((uintptr_t)work & 15) == 0 && ((uintptr_t)tile_plan & 15) == 0, "attention_plan: the plan's arrays must start on 16 bytes");
-    q6k_launch(attention_plan_kernel, 1, PLAN_THREADS, 0, st, positions, req_of_token, tile_tok0, tile_ntok, n_tiles, window, n_work, min_per,
+    q6k_launch(attention_plan_kernel, 1, PLAN_THREADS, 0, st, positions, req_of_token, tile_tok0, tile_ntok, n_tiles, window, chunk, n_work, min_per,
                work, tile_plan);
     return q6k_check_launch("attention_plan");
 }
@@ -977,7 +977,7 @@ Q6K_API int q6k_attention_mma_prepares(int hd, int G, int rows, int rotary_dim, 
 
 Q6K_API int q6k_attention_mma(const void* q, const void* k_pages, const void* v_pages, long long num_pages, const int* block_table,
                               int max_blocks, int page_size, const int* work, const int* tile_plan, int n_work, int n_tiles, int rows,
-                              int window, const float* sinks, float scale, void* out, float* part_o, float* part_ml, int Hq, int Hkv,
+                              int window, int chunk, const float* sinks, float scale, void* out, float* part_o, float* part_ml, int Hq, int Hkv,
                               int hd, int early, const float* qkv, int qkv_ld, int qkv_splits, long long qkv_split_stride, const float* q_norm, const float* k_norm, float eps,
                               const float* inv_freq, int rotary_dim, int write_kv, cudaStream_t st) {
     if (n_tiles == 0) return 0;
@@ -985,7 +985,7 @@ Q6K_API int q6k_attention_mma(const void* q, const void* k_pages, const void* v_
     const int G = Hq / Hkv;
     Q6K_REQUIRE(rows == 8 || rows == 16 || rows == 128, "attention_mma: tiles of %d rows (8, 16 or 128 are built)", rows);
     Q6K_REQUIRE(q6k_attention_mma_supported(hd, G, rows == 128) && G <= rows, "attention_mma: head_dim %d / group size %d is not covered by tiles of %d rows", hd, G, rows);
-    Q6K_REQUIRE(page_size > 0 && max_blocks > 0 && window >= 0 && n_work >= n_tiles && work && tile_plan,
+    Q6K_REQUIRE(page_size > 0 && max_blocks > 0 && window >= 0 && chunk >= 0 && n_work >= n_tiles && work && tile_plan,
                 "attention_mma: bad page_size %d / max_blocks %d / window %d / %d work items for %d tiles", page_size, max_blocks, window, n_work, n_tiles);
     Q6K_REQUIRE(n_work == n_tiles || (part_o && part_ml), "attention_mma: splitting the keys needs the partial buffers");
     Q6K_REQUIRE(Hkv <= 65535 && n_tiles <= 65535, "attention_mma: grid limit exceeded (Hkv=%d, tiles=%d)", Hkv, n_tiles);
@@ -994,7 +994,7 @@ Q6K_API int q6k_attention_mma(const void* q, const void* k_pages, const void* v_
     p.block_table = block_table, p.sinks = sinks, p.out = (__nv_bfloat16*)out;
     p.work = work, p.tile_plan = tile_plan, p.n_work = n_work;
     p.part_o = part_o, p.part_ml = part_ml;
-    p.max_blocks = max_blocks, p.page_size = page_size, p.window = window, p.Hq = Hq, p.Hkv = Hkv, p.G = G;
+    p.max_blocks = max_blocks, p.page_size = page_size, p.window = window, p.chunk = chunk, p.Hq = Hq, p.Hkv = Hkv, p.G = G;
     p.scale_log2 = scale * LOG2E;
     p.early = early;
     if (qkv) {

@@ -48,7 +48,7 @@ struct TcAttnParams {
     const int* tile_ntok;
     const float* sinks;                      // [Hq] or null
     __nv_bfloat16* out;                      // [T, Hq*HD]
-    int max_blocks, page_size, window, Hq, Hkv, G, pool_rows, num_pages;
+    int max_blocks, page_size, window, chunk, Hq, Hkv, G, pool_rows, num_pages;
     float scale_log2;
 };
 
@@ -202,7 +202,7 @@ __global__ void __launch_bounds__(TC_THREADS) attention_tc_kernel(const __grid_c
     for (int h = 0; h < 2; ++h) {
         pf[h] = nt_h[h] > 0 ? p.positions[h == 0 ? tok_h0 : tok_h1] : 0;
         pl[h] = pf[h] + nt_h[h] - 1;
-        lo_h[h] = p.window > 0 ? max(0, pf[h] - p.window + 1) : 0;
+        lo_h[h] = q6k_first_seen(pf[h], p.window, p.chunk);
         first_h[h] = nt_h[h] > 0 ? lo_h[h] / BN : 0;
         end_h[h] = nt_h[h] > 0 ? pl[h] / BN + 1 : 0;
     }
@@ -390,8 +390,8 @@ __global__ void __launch_bounds__(TC_THREADS) attention_tc_kernel(const __grid_c
         const int tt = row / G, hg = row % G;
         const bool row_valid = tt < ntk;
         const int pos = pf[h] + tt;
-        const int lim_hi = row_valid ? pos : -1, lim_lo = p.window > 0 ? pos - p.window + 1 : 0;
-        const int n_mine = end_h[h] - first_h[h];
+        const int lim_hi = row_valid ? pos : -1, lim_lo = q6k_first_seen(pos, p.window, p.chunk);
+        const int n_mine = end_h[h] - first_h[h], seen_by_all = q6k_first_seen(pl[h], p.window, p.chunk);
         float m = -INFINITY, l = 0.0f;
         bool ok = true;
         for (int t = 0; t < n_mine; ++t) {
@@ -404,8 +404,8 @@ __global__ void __launch_bounds__(TC_THREADS) attention_tc_kernel(const __grid_c
                 break;
             }
             tc_fence_after();
-            // tiles that every row of the half sees whole (below the diagonal, inside the window) need no mask
-            const bool whole = j0 + BN - 1 <= pf[h] && (p.window == 0 || j0 >= pl[h] - p.window + 1);
+            // tiles that every row of the half sees whole (below the diagonal, inside the window and the chunk) need no mask
+            const bool whole = j0 + BN - 1 <= pf[h] && j0 >= seen_by_all;
             // the row's 128 scores come into registers with one wait; masked ones become -inf
             float v[BN];
 #pragma unroll
@@ -587,16 +587,16 @@ Q6K_API int q6k_attention_tc_supported(int hd, int G, int page_size) {
 // [n_tiles, 2], for each CTA two tiles of one request, each of at most q6k_attention_tc_tile_tokens(G)
 // tokens at consecutive positions (the second may have no tokens); tiles whose key ranges overlap
 // share the K/V stream (for causal attention without a window: a late tile with an early one); out: bfloat16 [T, Hq*128].  Every tile reads its whole
-// key range (no key splits): the kernel for prompt portions.
+// key range (no key splits): the kernel for prompt portions.  window, chunk: what hides earlier keys (0: nothing), see q6k_first_seen.
 Q6K_API int q6k_attention_tc(const void* q, const void* k_pages, const void* v_pages, long long num_pages, const int* block_table,
                              int max_blocks, int page_size, const int* req_of_token, const int* positions, const int* tile_tok0,
-                             const int* tile_ntok, int n_tiles, int window, const float* sinks, float scale, void* out, int Hq, int Hkv,
+                             const int* tile_ntok, int n_tiles, int window, int chunk, const float* sinks, float scale, void* out, int Hq, int Hkv,
                              int hd, cudaStream_t st) {
     if (n_tiles == 0) return 0;
     Q6K_REQUIRE(Hq > 0 && Hkv > 0 && Hq % Hkv == 0, "attention_tc: bad head counts Hq=%d Hkv=%d", Hq, Hkv);
     const int G = Hq / Hkv;
     Q6K_REQUIRE(q6k_attention_tc_supported(hd, G, page_size), "attention_tc: head_dim %d / group size %d / page size %d is not covered", hd, G, page_size);
-    Q6K_REQUIRE(max_blocks > 0 && window >= 0 && n_tiles <= 65535, "attention_tc: bad max_blocks %d / window %d / %d tiles", max_blocks, window, n_tiles);
+    Q6K_REQUIRE(max_blocks > 0 && window >= 0 && chunk >= 0 && n_tiles <= 65535, "attention_tc: bad max_blocks %d / window %d / chunk %d / %d tiles", max_blocks, window, chunk, n_tiles);
     const long long pool_rows = num_pages * Hkv * page_size;
     Q6K_REQUIRE(pool_rows < (1LL << 31) && ((uintptr_t)k_pages & 15) == 0 && ((uintptr_t)v_pages & 15) == 0 && ((uintptr_t)q & 15) == 0 &&
                     ((uintptr_t)out & 15) == 0,
@@ -604,7 +604,7 @@ Q6K_API int q6k_attention_tc(const void* q, const void* k_pages, const void* v_p
     TcAttnParams p{};
     p.q = (const __nv_bfloat16*)q, p.block_table = block_table, p.req_of_token = req_of_token, p.positions = positions;
     p.tile_tok0 = tile_tok0, p.tile_ntok = tile_ntok, p.sinks = sinks, p.out = (__nv_bfloat16*)out;
-    p.max_blocks = max_blocks, p.page_size = page_size, p.window = window, p.Hq = Hq, p.Hkv = Hkv, p.G = G;
+    p.max_blocks = max_blocks, p.page_size = page_size, p.window = window, p.chunk = chunk, p.Hq = Hq, p.Hkv = Hkv, p.G = G;
     p.pool_rows = (int)pool_rows, p.num_pages = (int)num_pages, p.scale_log2 = scale * LOG2E;
     CUtensorMap tk, tv, tk_run, tv_run;
     const int box = page_size < 64 ? page_size : 64;       // pages of 128 keys are fetched as two boxes of 64

@@ -43,6 +43,13 @@ __device__ __forceinline__ float warp_max(float v) {
     for (int o = 16; o > 0; o >>= 1) v = fmaxf(v, __shfl_xor_sync(0xffffffffu, v, o));
     return v;
 }
+// The first key a query at position `pos` sees: all (window 0, chunk 0), the last `window` ones, those of its own block of `chunk`
+// positions (blocks counted from position 0), or what both leave.
+__device__ __forceinline__ int q6k_first_seen(int pos, int window, int chunk) {
+    int lo = window > 0 ? max(0, pos - window + 1) : 0;
+    if (chunk > 0) lo = max(lo, pos / chunk * chunk);
+    return lo;
+}
 // Sum over the block in a fixed order (warp results added in warp order); every thread gets it.
 // `red` holds at least 32 floats.  Safe to call repeatedly.
 __device__ __forceinline__ float block_sum(float v, float* red) {

@@ -657,13 +657,14 @@ def attention_tc_tile_tokens(G: int) -> int:
 def attention_tc(q: torch.Tensor, k_pages: torch.Tensor, v_pages: torch.Tensor, block_table: torch.Tensor,
                  req_of_token: torch.Tensor, positions: torch.Tensor, tile_tok0: torch.Tensor, tile_ntok: torch.Tensor,
                  window: Optional[int], sinks: Optional[torch.Tensor], scale: Optional[float] = None,
-                 out: Optional[torch.Tensor] = None) -> torch.Tensor:
+                 out: Optional[torch.Tensor] = None, chunk: Optional[int] = None) -> torch.Tensor:
     """bfloat16 attention for prompt portions with both products on tcgen05 tensor cores
     (accumulators and probabilities in tensor memory, K/V pages by TMA).  Head size 128.
     tile_tok0 / tile_ntok: [n, 2], two tiles of one request per CTA (StepContext.query_tile_pairs),
     each of at most attention_tc_tile_tokens(G) tokens at consecutive positions; the second may be
     empty.  Each tile reads its whole key range; the two share the K/V stream.  Only the rows of
-    the listed tiles are written (into `out` [T, Hq*hd] when given)."""
+    the listed tiles are written (into `out` [T, Hq*hd] when given).  chunk: a position sees the earlier keys of its own block
+    of `chunk` positions only."""
     _need(q, "q", torch.bfloat16)
     T, Hq, hd = q.shape
     _need(k_pages, "k_pages", torch.bfloat16)
@@ -684,7 +685,7 @@ def attention_tc(q: torch.Tensor, k_pages: torch.Tensor, v_pages: torch.Tensor, 
         _need(out, "out", torch.bfloat16, (T, Hq * hd))
     _call("q6k_attention_tc", _ptr(q), _ptr(k_pages), _ptr(v_pages), _ll(num_pages), _ptr(block_table),
           _i(block_table.shape[1]), _i(page_size), _ptr(req_of_token), _ptr(positions), _ptr(tile_tok0), _ptr(tile_ntok),
-          _i(tile_tok0.shape[0]), _i(window or 0), _ptr(sinks), _f(scale if scale is not None else 1.0 / math.sqrt(hd)), _ptr(out),
+          _i(tile_tok0.shape[0]), _i(window or 0), _i(chunk or 0), _ptr(sinks), _f(scale if scale is not None else 1.0 / math.sqrt(hd)), _ptr(out),
           _i(Hq), _i(Hkv), _i(hd), _stream())
     return out
 
@@ -724,12 +725,12 @@ def attention_mma_resident_ctas(hd: int, rows: int) -> int:
 
 
 def attention_plan(positions: torch.Tensor, req_of_token: torch.Tensor, tile_tok0: torch.Tensor, tile_ntok: torch.Tensor,
-                   window: Optional[int], n_work: int, min_per: int = 2, into=None):
+                   window: Optional[int], n_work: int, min_per: int = 2, into=None, chunk: Optional[int] = None):
     """Which CTA of attention_mma walks which key tiles, made on the device from the step's
     positions: (work int32 [n_work, 8], tile_plan int32 [n_tiles, 4]).  n_work (at least the number
     of tiles) CTAs per KV head share the key tiles about evenly; a tile's keys are split into
     parts of at least min_per key tiles (of 64 keys).  One plan serves every layer with this
-    window; recorded into a CUDA graph it is remade from the positions of each replay.
+    window and chunk; recorded into a CUDA graph it is remade from the positions of each replay.
     into: the pair of tensors of an earlier call with the same sizes, to be filled again."""
     for nm, t in (("req_of_token", req_of_token), ("positions", positions), ("tile_tok0", tile_tok0), ("tile_ntok", tile_ntok)):
         _need(t, nm, torch.int32)
@@ -742,7 +743,7 @@ def attention_plan(positions: torch.Tensor, req_of_token: torch.Tensor, tile_tok
     else:
         work = torch.empty((n_work, 8), dtype=torch.int32, device=positions.device)
         tile_plan = torch.empty((n_tiles, 4), dtype=torch.int32, device=positions.device)
-    _call("q6k_attention_plan", _ptr(positions), _ptr(req_of_token), _ptr(tile_tok0), _ptr(tile_ntok), _i(n_tiles), _i(window or 0),
+    _call("q6k_attention_plan", _ptr(positions), _ptr(req_of_token), _ptr(tile_tok0), _ptr(tile_ntok), _i(n_tiles), _i(window or 0), _i(chunk or 0),
           _i(n_work), _i(min_per), _ptr(work), _ptr(tile_plan), _stream())
     return work, tile_plan
 
@@ -760,11 +761,11 @@ def attention_mma(q: Optional[torch.Tensor], k_pages: torch.Tensor, v_pages: tor
                   req_of_token: torch.Tensor, positions: torch.Tensor, tile_tok0: torch.Tensor, tile_ntok: torch.Tensor,
                   rows: int, window: Optional[int], sinks: Optional[torch.Tensor], max_splits: int = 1, min_tiles: int = 2,
                   scale: Optional[float] = None, out: Optional[torch.Tensor] = None, plan=None, plan_is_old: bool = False,
-                  prepare=None) -> torch.Tensor:
+                  prepare=None, chunk: Optional[int] = None) -> torch.Tensor:
     """bfloat16 tensor-core attention over the pages.  Tiles: tile_tok0[i] is the first row and
     tile_ntok[i] the number of tokens (consecutive positions of one request, at most rows // G;
-    rows: 8, 16 or 128, see attention_mma_tile_rows) of tile i.  plan: attention_plan(...) of these tiles and this
-    window; without one it is made here for max_splits CTAs per tile on average, none with fewer
+    rows: 8, 16 or 128, see attention_mma_tile_rows) of tile i.  plan: attention_plan(...) of these tiles, this
+    window and chunk; without one it is made here for max_splits CTAs per tile on average, none with fewer
     than min_tiles key tiles.  Only the rows of the listed tiles are written (into `out`
     [T, Hq*hd] when given).  plan_is_old: the caller's word that the plan and the block table were
     made before the kernel launched just before this call (the one that writes this step's q and
@@ -812,7 +813,7 @@ def attention_mma(q: Optional[torch.Tensor], k_pages: torch.Tensor, v_pages: tor
     n_tiles = tile_tok0.numel()
     if plan is None:
         plan_is_old = False
-        plan = attention_plan(positions, req_of_token, tile_tok0, tile_ntok, window, n_tiles * max(1, max_splits), min_tiles)
+        plan = attention_plan(positions, req_of_token, tile_tok0, tile_ntok, window, n_tiles * max(1, max_splits), min_tiles, chunk=chunk)
     work, tile_plan = plan
     _need(work, "work", torch.int32)
     _need(tile_plan, "tile_plan", torch.int32, (n_tiles, 4))
@@ -829,7 +830,7 @@ def attention_mma(q: Optional[torch.Tensor], k_pages: torch.Tensor, v_pages: tor
         part_ml = ws[part_rows * hd: part_rows * (hd + 2)]
     _call("q6k_attention_mma", _ptr(q), _ptr(k_pages), _ptr(v_pages), _ll(num_pages), _ptr(block_table),
           _i(block_table.shape[1]), _i(page_size), _ptr(work), _ptr(tile_plan), _i(n_work), _i(n_tiles), _i(rows),
-          _i(window or 0), _ptr(sinks), _f(scale if scale is not None else 1.0 / math.sqrt(hd)), _ptr(out), _ptr(part_o), _ptr(part_ml),
+          _i(window or 0), _i(chunk or 0), _ptr(sinks), _f(scale if scale is not None else 1.0 / math.sqrt(hd)), _ptr(out), _ptr(part_o), _ptr(part_ml),
           _i(Hq), _i(Hkv), _i(hd), _i(1 if plan_is_old else 0), _ptr(qkv), _i(ld), _i(splits), _ll(split_stride), _ptr(q_norm), _ptr(k_norm), _f(eps),
           _ptr(inv_freq), _i(rotary_dim), _i(1 if write else 0), _stream())
     return out

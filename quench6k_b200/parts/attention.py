@@ -5,7 +5,8 @@ operations, crates/cuda/kernels/flint.cu:125-173 and :211-561 for the arithmetic
 Beyond the reference: values of another width than the keys (v_dim), a given score scale, a mask of chunks (a position
 sees the earlier positions of its own block of `chunk` positions, blocks counted from position 0), and the heads'
 softmax weights mixed by a learned [heads, heads] matrix before they meet the values (`talk`).  Layers that use any of
-these run the flexible attention kernels; the others run as before.  Two more options change what enters the attention,
+these run the flexible attention kernels; the others run as before.  Layers that use chunks alone run the others' tensor-core
+kernels too, for the head sizes those cover.  Two more options change what enters the attention,
 not the attention: biases on the q, k and v projections, and a short causal convolution over time on every channel of
 the projected q, k and v (before normalisation and rotation), whose last taps - 1 inputs are kept per request in a state
 slot so that a prompt may be cut anywhere.
@@ -76,6 +77,10 @@ class Attention(Mixer):
             raise ValueError("mixed heads are combined with neither sinks, maps nor a cap on the scores")
         self.flexible = (self.vd != head_dim or self.chunk is not None or self.talk or self.maps > 1 or self.softcap > 0.0
                          or head_dim % 16 != 0 or head_dim > 256)
+        # chunks alone (keys and values of one width, nothing else out of the ordinary): the fixed-shape tensor-core kernels take
+        # them for the head sizes they cover, the flexible kernels for the rest
+        self.only_chunks = (self.flexible and self.chunk is not None and self.vd == head_dim and not self.talk and self.maps == 1 and not self.softcap
+                            and head_dim % 16 == 0 and head_dim <= 256 and self.scale > 0.0)
         self.has_bias, self.taps = bool(bias), (int(conv) if conv else 0)
         if self.taps > 16:
             raise ValueError(f"{self.taps} convolution taps: the kernel takes 1 to 16")
@@ -232,7 +237,7 @@ class Attention(Mixer):
         return ops.short_conv(y, self.D, self._one_tap, self.o_bias, self._no_o_tail, ctx.req_of_token, ctx.q_start, ctx.slot_ids, ctx.R)
 
     def forward(self, xn, ctx, cache, state, out):
-        if self.flexible:
+        if self.flexible and not (self.only_chunks and self._fixed_shape(ctx)):
             return self._forward_flexible(xn, ctx, cache, state)
         rt = self.rt
         write = cache.write
@@ -276,6 +281,10 @@ class Attention(Mixer):
     prepare_in_attention = True   # the kernel that splits the keys makes q and the new keys itself where it can (else qk_prep does)
     tc_min_fill = 0.5             # the tcgen05 prompt kernel runs when its CTAs (two tiles each) cover at least this share of the SMs
 
+    def _fixed_shape(self, ctx) -> bool:
+        rt = self.rt
+        return not rt.is_fp32 and rt.tensor_cores and ops.attention_mma_tile_rows(self.hd, self.Hq // self.Hkv, ctx.max_q_len) > 0
+
     def _choose(self, cache, ctx):
         """("generic",) | ("split", plan args) | ("tc", tile pairs, plan args of the short requests or None): the tensor-core
         kernels for bfloat16 where they cover the head and group size, else the generic one.  The plans are made here."""
@@ -303,12 +312,12 @@ class Attention(Mixer):
         layers with this window."""
         tokens = rows // (self.Hq // self.Hkv)
         tok0, ntok, n_tiles = ctx.query_tiles(tokens, at_most)
-        key = ("attention_plan", tokens, at_most, self.window, self.Hkv)
+        key = ("attention_plan", tokens, at_most, self.window, self.chunk, self.Hkv)
         fresh = key not in ctx.made
         if fresh:                                   # the first layer of this pass with these tiles and this window
             ctx.plans[key] = ops.attention_plan(ctx.positions, ctx.req_of_token, tok0, ntok, self.window,
                                                 ops.attention_mma_resident_ctas(self.hd, rows) // self.Hkv, min_per=2,
-                                                into=ctx.plans.get(key))
+                                                into=ctx.plans.get(key), chunk=self.chunk)
             ctx.made.add(key)
         return rows, tok0, ntok, ctx.plans[key], fresh
 
@@ -318,7 +327,7 @@ class Attention(Mixer):
         if how[0] == "tc":
             (tok0, ntok), short = how[1], how[2]
             out = ops.attention_tc(q, cache.k, cache.v, table, ctx.req_of_token, ctx.positions, tok0, ntok, self.window,
-                                   self.sinks, scale=self.scale)
+                                   self.sinks, scale=self.scale, chunk=self.chunk)
             return out if short is None else self._split_keys(q, cache, table, ctx, short, out)
         return self._split_keys(q, cache, table, ctx, how[1])
 
@@ -331,7 +340,7 @@ class Attention(Mixer):
         # is surely complete.
         return ops.attention_mma(q, cache.k, cache.v, table, ctx.req_of_token, ctx.positions, tok0, ntok, rows, self.window,
                                  self.sinks, scale=self.scale, out=out, plan=plan, plan_is_old=prepare is None or not fresh,
-                                 prepare=prepare)
+                                 prepare=prepare, chunk=self.chunk)
 
     def _sm_count(self) -> int:
         if "_sms" not in self.__dict__:

@@ -107,9 +107,10 @@ def weights_of(z, chosen):
     return s / (s.sum() + 1e-20)
 
 
-def mixture(h, w, mlp, forced=None):
+def mixture(h, w, mlp, forced=None, identity=1.0):
     """Each token's chosen experts, weighted; an identity expert answers its input; plus the shared expert times one sigmoid
-    number per token.  forced [T, top]: use these experts instead of choosing.  Returns (result, chosen [T, top])."""
+    number per token.  forced [T, top]: use these experts instead of choosing.  identity: what an identity expert multiplies its
+    input by (tests that break it on purpose).  Returns (result, chosen [T, top])."""
     z = h @ w("router").T
     out = torch.zeros_like(h)
     all_chosen = []
@@ -121,7 +122,7 @@ def mixture(h, w, mlp, forced=None):
         all_chosen.append(chosen)
         for s in range(chosen.numel()):
             e = int(chosen[s])
-            answer = h[t] if e >= mlp["router"]["experts"] else expert(h[t], w(f"e{e}.gate"), w(f"e{e}.up"), w(f"e{e}.down"))
+            answer = identity * h[t] if e >= mlp["router"]["experts"] else expert(h[t], w(f"e{e}.gate"), w(f"e{e}.up"), w(f"e{e}.down"))
             out[t] = out[t] + wt[s] * answer
     if mlp.get("shared") is not None:
         out = out + torch.sigmoid(h @ w("shared.sg").T) * expert(h, w("shared.gate"), w("shared.up"), w("shared.down"))
@@ -146,10 +147,11 @@ def open_pass(x, x0, w_in, step):
     return torch.cat([x, x0], dim=-1) @ w_in.T + step
 
 
-def forward(cfg, weights, tokens, forced=None, layers_out=None, mixer=chunked_attention):
+def forward(cfg, weights, tokens, forced=None, layers_out=None, mixer=chunked_attention, ffn=mixture):
     """Logits [T, vocab] of one sequence.  forced: {executed position: [T, top]} experts to use in place of the router's
     choice.  forward.chosen holds the experts each routed position chose.  layers_out: a list that receives the stream
-    after every executed layer.  mixer: another function for the mixer (tests that break it on purpose)."""
+    after every executed layer.  mixer, ffn: other functions for the mixer and the feed-forward (tests that break them on
+    purpose)."""
     W = {k: v.to(F) for k, v in weights.items()}
     eps = cfg["norm"]["eps"]
     tok = torch.as_tensor(tokens, dtype=torch.long)
@@ -166,7 +168,7 @@ def forward(cfg, weights, tokens, forced=None, layers_out=None, mixer=chunked_at
             x = open_pass(x, x0, W["loop.in"], W["loop.step"][opens])
         x = x + norm(f"l{i}.norm1b", mixer(norm(f"l{i}.norm1", x), lambda n, i=i: W[f"l{i}.mix.{n}"], L["mixer"], eps))
         if L.get("mlp") is not None:
-            f, forward.chosen[p] = mixture(norm(f"l{i}.norm2", x), lambda n, i=i: W[f"l{i}.mlp.{n}"], L["mlp"], None if forced is None else forced.get(p))
+            f, forward.chosen[p] = ffn(norm(f"l{i}.norm2", x), lambda n, i=i: W[f"l{i}.mlp.{n}"], L["mlp"], None if forced is None else forced.get(p))
             x = x + norm(f"l{i}.norm2b", f)
         if layers_out is not None:
             layers_out.append(x.clone())
