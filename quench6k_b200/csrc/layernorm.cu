@@ -110,12 +110,24 @@ __device__ __forceinline__ float4 load4(const __nv_bfloat16* src) {
 // wait in shared memory, S of them at most MIX_SLOTS).
 constexpr int MIX_SLOTS = 64;
 
+// Sum over the 256 threads in a fixed order; `red` holds 8 floats that nothing else uses in this kernel.
+__device__ __forceinline__ float block_sum_once(float v, float* red) {
+    v = warp_sum(v);
+    if ((threadIdx.x & 31) == 0) red[threadIdx.x >> 5] = v;
+    __syncthreads();
+    float t = 0.0f;
+#pragma unroll
+    for (int i = 0; i < 8; ++i) t += red[i];
+    return t;
+}
+
 template <typename T, int V4, bool MIX>
 __global__ void __launch_bounds__(256) layernorm_reg_kernel(const LayerNormArgs a) {
     pdl_enter();
-    __shared__ float red[32];
+    __shared__ float red[4][8];
     __shared__ float slot_w[MIX ? MIX_SLOTS : 1];
     __shared__ int slot_row[MIX ? MIX_SLOTS : 1];
+    __shared__ int slots_live;
     const int r = blockIdx.x, D = a.D, t = a.rows ? a.rows[r] : r;
     const size_t at = (size_t)t * D;
     float* h = a.h + at;
@@ -124,12 +136,12 @@ __global__ void __launch_bounds__(256) layernorm_reg_kernel(const LayerNormArgs 
     bool has[V4];
 #pragma unroll
     for (int j = 0; j < V4; ++j) has[j] = (threadIdx.x + 256 * j) * 4 < D;
-    auto stats = [&](float& mean, float& inv) {
+    auto stats = [&](float& mean, float& inv, int which) {
         float s = 0.0f;
 #pragma unroll
         for (int j = 0; j < V4; ++j)
             if (has[j]) s += (v[j].x + v[j].y) + (v[j].z + v[j].w);
-        mean = block_sum(s, red) / (float)D;
+        mean = block_sum_once(s, red[which]) / (float)D;
         float q = 0.0f;
 #pragma unroll
         for (int j = 0; j < V4; ++j)
@@ -137,28 +149,50 @@ __global__ void __launch_bounds__(256) layernorm_reg_kernel(const LayerNormArgs 
                 const float a0 = v[j].x - mean, a1 = v[j].y - mean, a2 = v[j].z - mean, a3 = v[j].w - mean;
                 q += fmaf(a0, a0, a1 * a1) + fmaf(a2, a2, a3 * a3);
             }
-        inv = rsqrtf(block_sum(q, red) / (float)D + a.eps);
+        inv = rsqrtf(block_sum_once(q, red[which + 1]) / (float)D + a.eps);
     };
     float mean = 0.0f, inv = 1.0f;
+    // everything whose place is known is asked of memory before the first wait
+    float4 was[V4];
+#pragma unroll
+    for (int j = 0; j < V4; ++j)
+        if (has[j] && !(add && a.replace)) was[j] = load4(h + (threadIdx.x + 256 * j) * 4);
     if (add) {
         float gate = 1.0f, xw = 0.0f;
         int live = 0;
+#pragma unroll
+        for (int j = 0; j < V4; ++j) {
+            v[j] = make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+            if (has[j] && a.y) v[j] = load4(a.y + at + (threadIdx.x + 256 * j) * 4);
+        }
         if (MIX) {
             if (a.gate) gate = a.gate[t];
             if (a.x) xw = a.xw[t];
-            if (a.py && (int)threadIdx.x < a.S) {
-                slot_w[threadIdx.x] = a.pw[(size_t)t * a.S + threadIdx.x];
-                slot_row[threadIdx.x] = a.pair_row ? a.pair_row[(size_t)t * a.S + threadIdx.x] : t * a.S + threadIdx.x;
+            if (a.py) {
+                if (threadIdx.x < 32) {                      // the slots whose weight is not zero, in their order
+                    int n = 0;
+                    for (int s0 = 0; s0 < a.S; s0 += 32) {
+                        const int s = s0 + (int)threadIdx.x;
+                        const float g = s < a.S ? a.pw[(size_t)t * a.S + s] : 0.0f;
+                        const int place = s < a.S && a.pair_row ? a.pair_row[(size_t)t * a.S + s] : t * a.S + s;
+                        const unsigned on = __ballot_sync(0xffffffffu, g != 0.0f);
+                        if (g != 0.0f) {
+                            const int i = n + __popc(on & ((1u << threadIdx.x) - 1u));
+                            slot_w[i] = g, slot_row[i] = place;
+                        }
+                        n += __popc(on);
+                    }
+                    if (threadIdx.x == 0) slots_live = n;
+                }
+                __syncthreads();
+                live = slots_live;
             }
-            if (a.py) __syncthreads(), live = a.S;
         }
 #pragma unroll
         for (int j = 0; j < V4; ++j)
             if (has[j]) {
                 const int c = (threadIdx.x + 256 * j) * 4;
-                v[j] = make_float4(0.0f, 0.0f, 0.0f, 0.0f);
                 if (a.y) {
-                    v[j] = load4(a.y + at + c);
                     for (int k = 1; k < a.splits; ++k) {
                         const float4 o = load4(a.y + k * a.split_stride + at + c);
                         v[j].x += o.x, v[j].y += o.y, v[j].z += o.z, v[j].w += o.w;
@@ -167,9 +201,9 @@ __global__ void __launch_bounds__(256) layernorm_reg_kernel(const LayerNormArgs 
                 }
                 if (MIX) {
                     float4 sp = make_float4(0.0f, 0.0f, 0.0f, 0.0f);
-                    for (int s = 0; s < live; ++s) {
+#pragma unroll 4
+                    for (int s = 0; s < live; ++s) {         // four rows' loads on the way at a time
                         const float g = slot_w[s];
-                        if (g == 0.0f) continue;
                         const float4 o = load4(a.py + (size_t)slot_row[s] * D + c);
                         sp.x = fmaf(g, o.x, sp.x), sp.y = fmaf(g, o.y, sp.y), sp.z = fmaf(g, o.z, sp.z), sp.w = fmaf(g, o.w, sp.w);
                     }
@@ -180,21 +214,21 @@ __global__ void __launch_bounds__(256) layernorm_reg_kernel(const LayerNormArgs 
                     }
                 }
             }
-        if (!a.replace) stats(mean, inv);
+        if (!a.replace) stats(mean, inv, 0);
     }
 #pragma unroll
     for (int j = 0; j < V4; ++j)
         if (has[j]) {
             const int c = (threadIdx.x + 256 * j) * 4;
             if (!add) {
-                v[j] = load4(h + c);
+                v[j] = was[j];
             } else if (a.replace) {
                 if (a.vec) {
                     const float4 e = load4(a.vec + c);
                     v[j].x += e.x, v[j].y += e.y, v[j].z += e.z, v[j].w += e.w;
                 }
             } else {
-                const float4 hv = load4(h + c), ww = load4(a.wa + c), bb = load4(a.ba + c);
+                const float4 hv = was[j], ww = load4(a.wa + c), bb = load4(a.ba + c);
                 v[j].x = hv.x + ((v[j].x - mean) * inv * ww.x + bb.x), v[j].y = hv.y + ((v[j].y - mean) * inv * ww.y + bb.y);
                 v[j].z = hv.z + ((v[j].z - mean) * inv * ww.z + bb.z), v[j].w = hv.w + ((v[j].w - mean) * inv * ww.w + bb.w);
             }
@@ -206,7 +240,7 @@ __global__ void __launch_bounds__(256) layernorm_reg_kernel(const LayerNormArgs 
         }
     if (!a.out) return;
     T* o = (T*)a.out + (size_t)r * a.ldo;
-    if (a.w) stats(mean, inv);
+    if (a.w) stats(mean, inv, 2);
 #pragma unroll
     for (int j = 0; j < V4; ++j)
         if (has[j]) {

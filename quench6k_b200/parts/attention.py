@@ -81,6 +81,8 @@ class Attention(Mixer):
         # them for the head sizes they cover, the flexible kernels for the rest
         self.only_chunks = (self.flexible and self.chunk is not None and self.vd == head_dim and not self.talk and self.maps == 1 and not self.softcap
                             and head_dim % 16 == 0 and head_dim <= 256 and self.scale > 0.0)
+        if self.only_chunks:
+            self.tc_min_fill = 0.15      # a chunk bounds the keys of a tile, so the prompt kernel pays from fewer tiles on
         self.has_bias, self.taps = bool(bias), (int(conv) if conv else 0)
         if self.taps > 16:
             raise ValueError(f"{self.taps} convolution taps: the kernel takes 1 to 16")
